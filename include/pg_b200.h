@@ -403,7 +403,8 @@ int pg_moe_combine(float* x, const void* y, int ldy, const int32_t* pair_pos, co
 enum {
   PG_GLU_NONE = 0,
   PG_GLU_SILU = 1,    /* silu(g) * u */
-  PG_GLU_CLAMPED = 2  /* g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1) */
+  PG_GLU_CLAMPED = 2, /* g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1) */
+  PG_ACT_RELU2 = 3    /* pg_moe_gemm_act only: ONE product per output (W_e is [N][K]), max(z, 0)^2 before the rounding */
 };
 
 /* pg_moe_gemm with the pairing given by name (pg_moe_gemm: swiglu != 0 is PG_GLU_SILU). */
@@ -561,6 +562,67 @@ int pg_gate_groupnorm(void* out, int ld_out, const float* y, const void* z, int 
                       int groups, float eps, int dtype, void* stream);
 int pg_lightning_attention_ex(float* out, float* state, const float* rec, const float* decay, const float* skip,
                               const int32_t* segs, int n_segs, int heads, int dim, int vdim, void* stream);
+
+/* ---- layer norms between sublayers, experts picked by token id, retention, capped attention over tied values -------
+ * pg_residual_layernorm: the whole step from one sublayer's output to the next one's operand, per row r of the fp32
+ *   stream x [.., D] (src = rows_idx ? rows_idx[r] : r):
+ *     x = table[ids[src]] (PG_EMB_INIT: x is not read) ; x += y[src] (dense rows, y_pos NULL) or
+ *     y_w * sum_k y[y_pos[src * y_top + k]] (expert rows; a negative place adds nothing) ;
+ *     x += table[ids[src]] (PG_EMB_ADD) ; x += vec (model dtype, may be NULL) ; written back unless rows_idx is given ;
+ *     out = ((x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b) * out_scale, rounded once (out NULL: the sum alone).
+ *   Without out_pos row r goes to out[r], with it to the rows out[out_pos[r * out_top + k]] (negative: dropped).  An id
+ *   outside [0, vocab) counts as a zero row and sets *err_flag to 1.
+ * pg_cache_append: columns [k_col0, k_col0 + cols) of the projection rows, unchanged, to the pool rows of
+ *   (tok_slot, tok_pos).
+ * pg_moe_table_sort: routing by tables of expert indices per token id: the pairs of all n_layers layers are grouped by
+ *   expert in one launch.  desc [n_layers][5] = {first entry of the layer's [vocab][top] table in `tables`, experts, top,
+ *   sum of the earlier layers' top, sum of the earlier layers' (experts + 1)}; layer l's pair_pos (place of pair t * top + k
+ *   in expert order, -1 for an id outside the vocabulary) starts at n_tokens * desc[l][3], its offsets [experts + 1] at
+ *   desc[l][4].
+ * pg_retention_prep: records of pg_lightning_attention from the fused projection: the first rot_dims columns of every q
+ *   and k head are rotated by tok_pos * freq (freq: device (high, low) float pairs, rot_dims / 2 of them; column i with
+ *   i + rot_dims / 2, or 2i with 2i + 1 when interleaved != 0), k is multiplied by k_scale after it, v passes; fp32.
+ * pg_headnorm_gate_ex: pg_headnorm_gate with the gate through silu instead of the sigmoid (gate_silu != 0); w may be NULL.
+ * pg_attention_ragged_capped: pg_attention_ragged_masked with a query temperature (temp_every > 0: q . k of a query at
+ *   position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)) and a softcap (> 0: score <-
+ *   softcap * tanh(score / softcap), right after scale and temperature).  k_pool and v_pool may be the same pool.
+ * pg_attention_ragged_tc_capped: the same on the tcgen05 kernel (a temperature needs a cap there).  Head sizes that are
+ *   multiples of 8 up to 256 (pg_attention_ragged_tc_ok8); with the values in the key rows of one pool nothing is
+ *   loaded twice. */
+enum { PG_EMB_NONE = 0, PG_EMB_INIT = 1, PG_EMB_ADD = 2 };
+int pg_residual_layernorm(void* out, int ld_out, float* x, const void* y, int ldy, const int32_t* y_pos, int y_top,
+                          float y_w, const int64_t* ids, const void* table, long long vocab, int emb_mode,
+                          const void* vec, const void* w, const void* b, float eps, float out_scale,
+                          const int32_t* rows_idx, const int32_t* out_pos, int out_top, int rows, int D,
+                          int* err_flag, int dtype, void* stream);
+int pg_cache_append(void* pool, int ld_pool, const void* proj, int ld, int k_col0, int cols, const int32_t* page_table,
+                    int pt_stride, int page_size, const int32_t* tok_slot, const int32_t* tok_pos, int n_tokens,
+                    int dtype, void* stream);
+int pg_moe_table_sort(int32_t* offsets, int32_t* pair_pos, const int32_t* tables, const int32_t* desc, int n_layers,
+                      const int64_t* ids, int n_tokens, long long vocab, int max_experts, void* stream);
+int pg_retention_prep(float* rec, const void* proj, int ld, int q_col0, int k_col0, int v_col0, const float* freq,
+                      int rot_dims, int interleaved, float k_scale, const int32_t* tok_pos, int n_tokens, int heads,
+                      int dim, int vdim, int dtype, void* stream);
+int pg_headnorm_gate_ex(void* out, int ld_out, const float* o, const void* w, const void* gate, int ld_gate,
+                        int gate_silu, int n_tokens, int heads, int dim, float eps, float out_scale, int dtype,
+                        void* stream);
+int pg_attention_ragged_capped(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,
+                               int gate_per_head, const void* k_pool, int ld_k, const void* v_pool, int ld_v,
+                               const int32_t* page_table, int pt_stride, int page_size, const int32_t* tok_slot,
+                               const int32_t* tok_pos, int n_tokens, int n_heads, int n_kv_heads, int dim, int vdim,
+                               float scale, int window, int keep_first, int chunk, const float* slopes,
+                               int sigmoid_weights, const float* head_bias, const float* sink, float softcap,
+                               float temp_coef, int temp_every, const float* out_rot, int out_rot_interleaved,
+                               float out_scale, float* ws, long long ws_floats, int dtype, void* stream);
+int pg_attention_ragged_tc_ok8(int dim, int vdim, int page_size, int ld_q, int ld_out, int ld_gate, int dtype);
+int pg_attention_ragged_tc_capped(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,
+                                  int gate_per_head, const void* k_pool, int ld_k, const void* v_pool, int ld_v,
+                                  long long pool_rows, const int32_t* page_table, int pt_stride, int page_size,
+                                  const int32_t* tiles, int n_tiles, int n_tokens, int n_heads, int n_kv_heads, int dim,
+                                  int vdim, float scale, int window, int keep_first, int chunk, const float* slopes,
+                                  int sigmoid_weights, const float* head_bias, const float* sink, float softcap,
+                                  float temp_coef, int temp_every, const float* out_rot, int out_rot_interleaved,
+                                  float out_scale, int* err_flag, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -12,6 +12,9 @@
 // [0, min(keep_first, lo)) ++ [lo, p], which every kernel below walks through one index map.  weights == 1 replaces
 // the softmax by unnormalised weights sigmoid(score + head_bias[h]).  The gate is either one value per output column
 // (gate_per_head == 0) or one per (token, head); the result is multiplied by out_scale before the single rounding.
+// pg_attention_ragged_capped adds, both in fp32: a query temperature (the score of a query at position p is multiplied by
+// 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)) and a softcap (score <- softcap * tanh(score / softcap), after the
+// scale and before distance bias and head bias).  Key and value pool may be one and the same (the values are the keys).
 // pg_attention_ragged_sink adds: sink[h], a per-head logit without key or value whose exp joins the softmax
 // denominator once (after all partial sums are merged), and explicit row strides of the key and the value pool, so
 // that the value rows may be a prefix of the key rows of ONE pool (latent attention: key [c | k_rot], value c).
@@ -105,7 +108,17 @@ struct RagAttnParams {
   int chunk;                     // > 0: a key is visible only inside the query's block of `chunk` positions
   const float* out_rot;          // [vdim / 2]: the result is turned back by -position * out_rot[m] (rotated values)
   int out_rot_interleaved;       // pairs (2m, 2m + 1) instead of (m, m + vdim / 2)
+  float softcap;                 // > 0: score <- softcap * tanh(score / softcap)
+  float temp_coef; int temp_every;   // query temperature 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)
 };
+
+// The factor of q . k for a query at position pos.
+__device__ __forceinline__ float query_scale(const RagAttnParams& p, int pos) {
+  return p.temp_every > 0 ? p.scale * (1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1))) : p.scale;
+}
+__device__ __forceinline__ float capped(const RagAttnParams& p, float s) {
+  return p.softcap > 0.f ? p.softcap * tanhf(s / p.softcap) : s;
+}
 
 // The visible keys of a token at position pos as one list: n_keep kept first positions, then [lo, pos].
 struct KeyRange {
@@ -122,8 +135,8 @@ struct KeyRange {
 // Process keys [lo, hi] (inclusive) of one (token, head) for the calling warp; (m, l, acc) are the running state.
 template <typename T, int DPL>
 __device__ __forceinline__ void attend_range(const RagAttnParams& p, const float* qs, const int32_t* pt_row, int g,
-                                             int pos, float slope, float bias, const KeyRange& kr, float& m, float& l,
-                                             float* acc) {
+                                             int pos, float qscale, float slope, float bias, const KeyRange& kr, float& m,
+                                             float& l, float* acc) {
   const int lo = 0, hi = kr.count - 1;              // virtual key indices
   const int lane = threadIdx.x & 31;
   const T* kpool = reinterpret_cast<const T*>(p.k_pool);
@@ -136,7 +149,7 @@ __device__ __forceinline__ void attend_range(const RagAttnParams& p, const float
     long long row = 0;
     if (valid) {
       row = (long long)pt_row[j / p.page_size] * p.page_size + j % p.page_size;
-      s = dot_row<T>(qs, kpool + row * kw + g * p.dim, p.dim) * p.scale - slope * (float)(pos - j) + bias;
+      s = capped(p, dot_row<T>(qs, kpool + row * kw + g * p.dim, p.dim) * qscale) - slope * (float)(pos - j) + bias;
     }
     float m_new = m, pj;
     if (p.sigmoid_weights) {                       // unnormalised: no running maximum, m stays 0
@@ -248,7 +261,7 @@ __global__ void __launch_bounds__(256) attention_ragged_kernel(RagAttnParams p) 
   float m = p.sigmoid_weights ? 0.f : -INFINITY, l = 0.f, acc[DPL];
 #pragma unroll
   for (int i = 0; i < DPL; ++i) acc[i] = 0.f;
-  attend_range<T, DPL>(p, qs, pt_row, g, pos, slope, bias, kr, m, l, acc);
+  attend_range<T, DPL>(p, qs, pt_row, g, pos, query_scale(p, pos), slope, bias, kr, m, l, acc);
   store_out<T, DPL>(p, t, h, m, l, acc);
 }
 
@@ -299,6 +312,7 @@ __global__ void __launch_bounds__(128) attention_ragged_split_kernel(RagAttnPara
   const int pos = p.tok_pos[t];
   const int32_t* pt_row = p.page_table + (size_t)p.tok_slot[t] * p.pt_stride;
   const KeyRange kr(pos, p.window, p.keep_first, p.chunk);
+  const float qscale = query_scale(p, pos);
   float slope[R], bias[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
@@ -331,7 +345,7 @@ __global__ void __launch_bounds__(128) attention_ragged_split_kernel(RagAttnPara
       row = (long long)pt_row[j / p.page_size] * p.page_size + j % p.page_size;
       dot_rows<T, R>(qs, p.dim, kpool + row * kw + g * p.dim, s);
 #pragma unroll
-      for (int r = 0; r < R; ++r) s[r] = s[r] * p.scale - slope[r] * (float)(pos - j) + bias[r];
+      for (int r = 0; r < R; ++r) s[r] = capped(p, s[r] * qscale) - slope[r] * (float)(pos - j) + bias[r];
     }
 #pragma unroll
     for (int r = 0; r < R; ++r) {
@@ -493,9 +507,25 @@ extern "C" int pg_attention_ragged_masked(void* out, int ld_out, const void* q, 
                                           int chunk, const float* slopes, int sigmoid_weights, const float* head_bias,
                                           const float* sink, const float* out_rot, int out_rot_interleaved,
                                           float out_scale, float* ws, long long ws_floats, int dtype, void* stream) {
+  return pg_attention_ragged_capped(out, ld_out, q, ld_q, gate, ld_gate, gate_per_head, k_pool, ld_k, v_pool, ld_v, page_table,
+                                    pt_stride, page_size, tok_slot, tok_pos, n_tokens, n_heads, n_kv_heads, dim, vdim, scale,
+                                    window, keep_first, chunk, slopes, sigmoid_weights, head_bias, sink, 0.f, 0.f, 0, out_rot,
+                                    out_rot_interleaved, out_scale, ws, ws_floats, dtype, stream);
+}
+
+extern "C" int pg_attention_ragged_capped(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,
+                                          int gate_per_head, const void* k_pool, int ld_k, const void* v_pool, int ld_v,
+                                          const int32_t* page_table, int pt_stride, int page_size,
+                                          const int32_t* tok_slot, const int32_t* tok_pos, int n_tokens, int n_heads,
+                                          int n_kv_heads, int dim, int vdim, float scale, int window, int keep_first,
+                                          int chunk, const float* slopes, int sigmoid_weights, const float* head_bias,
+                                          const float* sink, float softcap, float temp_coef, int temp_every,
+                                          const float* out_rot, int out_rot_interleaved, float out_scale, float* ws,
+                                          long long ws_floats, int dtype, void* stream) {
   if (n_tokens <= 0) return PG_OK;
   PG_REQUIRE(chunk >= 0 && (chunk == 0 || keep_first == 0), "attention_ragged: blocks of %d positions with %d kept first ones",
              chunk, keep_first);
+  PG_REQUIRE(softcap >= 0.f && temp_every >= 0, "attention_ragged: softcap %g, temperature steps of %d", (double)softcap, temp_every);
   if (ld_k <= 0) ld_k = n_kv_heads * dim;
   if (ld_v <= 0) ld_v = n_kv_heads * vdim;
   PG_REQUIRE(ld_k >= n_kv_heads * dim && ld_v >= n_kv_heads * vdim, "attention_ragged: pool rows of %d / %d elements", ld_k, ld_v);
@@ -505,7 +535,7 @@ extern "C" int pg_attention_ragged_masked(void* out, int ld_out, const void* q, 
   RagAttnParams p = {out, ld_out, q, ld_q, gate, ld_gate, k_pool, v_pool, page_table, pt_stride, page_size, tok_slot,
                      tok_pos, n_tokens, n_heads, n_kv_heads, dim, vdim, scale, window, slopes, keep_first,
                      sigmoid_weights ? 1 : 0, head_bias, gate_per_head ? 1 : 0, out_scale, ld_k, ld_v, sink, chunk, out_rot,
-                     out_rot_interleaved ? 1 : 0};
+                     out_rot_interleaved ? 1 : 0, softcap, temp_coef, temp_every};
   cudaStream_t st = (cudaStream_t)stream;
   const int dpl = (vdim + 31) / 32;
   PG_DISPATCH_DTYPE(dtype, T, {

@@ -14,6 +14,12 @@
 // window: the key tiles are then the pages that hold them (as far as they lie before the window's first page)
 // followed by the window's pages.  sigmoid_weights: ONE pass, p = sigmoid(s + head_bias[h]), no maximum, no sum.  The
 // gate may be one value per (token, head); the result is multiplied by out_scale before it is rounded.
+// pg_attention_ragged_tc_capped adds a query temperature and a softcap (both fp32, as in attention_ragged.cu; the kernel is
+// instantiated with and without the cap).  A capped score is bounded, so its softmax needs no maximum: with a cap of at
+// most 40 and bf16 weights (fp32's exponent range) the kernel runs ONE pass with p = exp(s - max(0, sink)), half the
+// MMAs of the two-pass form.  Head sizes are multiples of 8: the operand maps are {column, head, row} tensors, so the
+// 64-column tiles of a narrower head are filled up with zeros by the TMA unit.  When the value rows are the key rows (or a
+// prefix of them) of ONE pool, P V reads V from the K tile that S = Q K^T has just used and nothing is loaded twice.
 // Every mbarrier wait is bounded: a wait that gives up sets the error flag, the roles leave their loops, the CTA lets
 // its copies land, frees its TMEM and returns.
 #include <cmath>
@@ -60,17 +66,21 @@ struct WinParams {
   int chunk;                     // > 0: a key is visible only inside the query's block of `chunk` positions
   const float* out_rot;          // [vdim / 2]: the result is turned back by -position * out_rot[m] (rotated values)
   int out_rot_interleaved;       // pairs (2m, 2m + 1) instead of (m, m + vdim / 2)
+  float softcap;                 // > 0: score <- softcap * tanh(score / softcap)
+  float temp_coef; int temp_every;   // query temperature 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)
+  int tied;                      // the value row is (a prefix of) the key row: V is read from the K tile
+  int bounded;                   // capped scores that need no maximum: one pass
 };
 
-template <typename T>
+template <typename T, bool CAP>
 __global__ void __launch_bounds__(256, 1)
 attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                            const __grid_constant__ CUtensorMap map_v, WinParams p) {
   constexpr int FMT = std::is_same<T, bf16>::value ? 1 : 0;
-  const int KB = p.dim / 64, VB = p.vdim / 64;
-  const int Q_BYTES = WQ * p.dim * 2, K_BYTES = WK * p.dim * 2, V_BYTES = WK * p.vdim * 2, P_BYTES = WQ * WK * 2;
+  const int KB = (p.dim + 63) / 64, VB = (p.vdim + 63) / 64;          // 64-column tiles of a head, zero-filled behind it
+  const int Q_BYTES = WQ * KB * 128, K_BYTES = WK * KB * 128, V_BYTES = p.tied ? 0 : WK * VB * 128, P_BYTES = WQ * WK * 2;
   const int S_COL = 0, O_COL = WK;
-  const int tmem_cols = (WK + p.vdim <= 256) ? 256 : 512;
+  const int tmem_cols = (WK + VB * 64 <= 256) ? 256 : 512;
 
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -118,39 +128,39 @@ attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
   const int n_tiles = n_keep + hi / WK - t_lo + 1;
   auto page_of = [&](int t) { return t < n_keep ? t : t_lo + (t - n_keep); };   // key tile -> page of the sequence
   const int32_t* pt_row = p.page_table + (size_t)slot * p.pt_stride;
-  const bool sig = p.sigmoid_weights != 0;
+  const bool sig = p.sigmoid_weights != 0, one_pass = sig || (CAP && p.bounded);
 
   if (warp == 0 && lane == 0) {
     // ===================== TMA + MMA issuer (one thread) =====================
     const uint32_t idesc_s = umma_idesc(FMT, WQ, WK);
-    const uint32_t idesc_o = umma_idesc(FMT, WQ, p.vdim) | (1u << 16);  // B (= V) is MN-major
+    const uint32_t idesc_o = umma_idesc(FMT, WQ, VB * 64) | (1u << 16);            // B (= V) is MN-major
     mbar_expect_tx(bar_q, Q_BYTES);
     for (int kb = 0; kb < KB; ++kb)
-      tma_load_2d(s_q + kb * (WQ * 128), &map_q, bar_q, h * p.dim + kb * 64, row0);
-    const int total = sig ? n_tiles : 2 * n_tiles;
+      tma_load_3d(s_q + kb * (WQ * 128), &map_q, bar_q, kb * 64, h, row0);
+    const int total = one_pass ? n_tiles : 2 * n_tiles;
     auto request = [&](int i) {   // K of flat step i into K buffer i & 1
       const int t = page_of(i >= n_tiles ? i - n_tiles : i), bf = i & 1;
       const int row = pt_row[t] * WK;
       mbar_expect_tx(bar_kv(bf), K_BYTES);
       for (int kb = 0; kb < KB; ++kb)
-        tma_load_2d(s_k(bf) + kb * (WK * 128), &map_k, bar_kv(bf), kvh * p.dim + kb * 64, row);
+        tma_load_3d(s_k(bf) + kb * (WK * 128), &map_k, bar_kv(bf), kb * 64, kvh, row);
     };
     auto request_v = [&](int t) {   // V of key tile t (pass 1) into the V buffer
       const int row = pt_row[page_of(t)] * WK;
       mbar_expect_tx(bar_v, V_BYTES);
       for (int vb = 0; vb < VB; ++vb)
-        tma_load_2d(s_vb + vb * (WK * 128), &map_v, bar_v, kvh * p.vdim + vb * 64, row);
+        tma_load_3d(s_vb + vb * (WK * 128), &map_v, bar_v, vb * 64, kvh, row);
     };
     request(0);
     if (!wait_lim(bar_q, 0, fail)) goto issuer_done;
     for (int it = 0; it < total; ++it) {
-      const int pass = (sig || it >= n_tiles) ? 1 : 0, t = it >= n_tiles ? it - n_tiles : it, bf = it & 1;
+      const int pass = (one_pass || it >= n_tiles) ? 1 : 0, t = it >= n_tiles ? it - n_tiles : it, bf = it & 1;
       if (it > 0 && !wait_lim(bar_sfree, (it - 1) & 1, fail)) goto issuer_done;          // S of the previous tile was read
       if (pass == 1 && t > 0 && !wait_lim(bar_o, (t - 1) & 1, fail)) goto issuer_done;   // previous PV done with V and P
-      if (pass == 1) request_v(t);                                 // lands behind S(it) and the softmax of this tile
+      if (pass == 1 && !p.tied) request_v(t);                      // lands behind S(it) and the softmax of this tile
       if (!wait_lim(bar_kv(bf), (it >> 1) & 1, fail)) goto issuer_done;
       tc_fence_after();
-      for (int ks = 0; ks < p.dim / 16; ++ks) {                    // S = Q K^T
+      for (int ks = 0; ks < (p.dim + 15) / 16; ++ks) {             // S = Q K^T
         const uint32_t off_q = (ks / 4) * (WQ * 128) + (ks % 4) * 32, off_k = (ks / 4) * (WK * 128) + (ks % 4) * 32;
         umma(tmem_base + S_COL, umma_desc(s_q + off_q), umma_desc(s_k(bf) + off_k), idesc_s, ks > 0 ? 1u : 0u);
       }
@@ -158,10 +168,11 @@ attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
       if (it + 1 < total) request(it + 1);                         // the other K buffer is free (bar_sfree above)
       if (pass == 1) {
         if (!wait_lim(bar_p, t & 1, fail)) goto issuer_done;       // P tile is in shared memory
-        if (!wait_lim(bar_v, t & 1, fail)) goto issuer_done;       // and so is V
+        if (!p.tied && !wait_lim(bar_v, t & 1, fail)) goto issuer_done;   // and so is V
+        const uint32_t s_val = p.tied ? s_k(bf) : s_vb;            // a tied tile stays until the next tile's P V is over
         tc_fence_after();
         for (int ks = 0; ks < WK / 16; ++ks) {                     // O += P V
-          umma(tmem_base + O_COL, umma_desc(s_p + ks * 32), umma_desc_mn_w(s_vb + ks * 2048, WK * 128), idesc_o,
+          umma(tmem_base + O_COL, umma_desc(s_p + ks * 32), umma_desc_mn_w(s_val + ks * 2048, WK * 128), idesc_o,
                (t > 0 || ks > 0) ? 1u : 0u);
         }
         umma_commit(bar_o);
@@ -176,9 +187,13 @@ attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
     const float slope = p.slopes ? p.slopes[h] : 0.f, hbias = p.head_bias ? p.head_bias[h] : 0.f;
     const int blk0 = p.chunk > 0 ? i / p.chunk * p.chunk : 0;      // first position of this row's block
     float m = -INFINITY, l = 0.f;
+    if (CAP && p.bounded) m = p.sink ? fmaxf(p.sink[h], 0.f) : 0.f;  // any value near the scores does: they are bounded
+    float qscale = p.scale;
+    if (CAP && p.temp_every > 0) qscale *= 1.f + p.temp_coef * logf((float)((i + 1) / p.temp_every + 1));
+    const float cap_in = CAP ? 2.f * qscale / p.softcap : 0.f, cap_out = 2.f * p.softcap;
     int it = 0;
     bool ok = true;
-    for (int pass = sig ? 1 : 0; pass < 2 && ok; ++pass) {
+    for (int pass = one_pass ? 1 : 0; pass < 2 && ok; ++pass) {
       for (int t = 0; t < n_tiles; ++t, ++it) {
         if (!wait_lim(bar_s, it & 1, fail)) { ok = false; break; }
         tc_fence_after();
@@ -193,7 +208,10 @@ attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
           for (int jj = 0; jj < 32; ++jj) {
             const int j = j0 + c * 32 + jj, back = i - j;
             const bool vis = back >= 0 && j >= blk0 && (p.window <= 0 || back < p.window || j < p.keep_first);
-            s[jj] = vis ? s[jj] * p.scale - slope * (float)back + hbias : -INFINITY;
+            float sc = s[jj] * qscale;
+            if (CAP)           // cap * tanh(z / cap) = cap - 2 cap / (exp(2 z / cap) + 1): absolute error a few 1e-7 of the cap
+              sc = p.softcap - __fdividef(cap_out, __expf(s[jj] * cap_in) + 1.f);
+            s[jj] = vis ? sc - slope * (float)back + hbias : -INFINITY;
           }
           if (pass == 0) {
 #pragma unroll
@@ -234,6 +252,7 @@ attention_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
         if (r >= rows) return;
 #pragma unroll
         for (int q0 = 0; q0 < 32; q0 += 8) {
+          if (c * 32 + q0 >= p.vdim) break;                        // vdim is a multiple of 8
           float w[8], gt[8];
           if (grow) unpack<T>(*reinterpret_cast<const uint4*>(grow + c * 32 + q0), gt);
 #pragma unroll
@@ -319,6 +338,13 @@ extern "C" int pg_attention_ragged_tc_ok(int dim, int vdim, int page_size, int l
   return tc::encode_fn() != nullptr ? 1 : 0;
 }
 
+extern "C" int pg_attention_ragged_tc_ok8(int dim, int vdim, int page_size, int ld_q, int ld_out, int ld_gate, int dtype) {
+  static const int enabled = env_int("PG_RAGGED_ATTN_TC", 1);
+  if (!enabled || (dtype != PG_BF16 && dtype != PG_F16) || page_size != tc::WK) return 0;
+  if (dim % 8 || vdim % 8 || dim > 256 || vdim > 256 || ld_q % 8 || ld_out % 8 || ld_gate % 8) return 0;
+  return tc::encode_fn() != nullptr ? 1 : 0;
+}
+
 extern "C" int pg_attention_ragged_tc_sink(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,
                                            int gate_per_head, const void* k_pool, int ld_k, const void* v_pool, int ld_v,
                                            long long pool_rows, const int32_t* page_table, int pt_stride, int page_size,
@@ -340,6 +366,21 @@ extern "C" int pg_attention_ragged_tc_masked(void* out, int ld_out, const void* 
                                              const float* slopes, int sigmoid_weights, const float* head_bias,
                                              const float* sink, const float* out_rot, int out_rot_interleaved,
                                              float out_scale, int* err_flag, int dtype, void* stream) {
+  return pg_attention_ragged_tc_capped(out, ld_out, q, ld_q, gate, ld_gate, gate_per_head, k_pool, ld_k, v_pool, ld_v, pool_rows,
+                                       page_table, pt_stride, page_size, tiles, n_tiles, n_tokens, n_heads, n_kv_heads, dim,
+                                       vdim, scale, window, keep_first, chunk, slopes, sigmoid_weights, head_bias, sink, 0.f,
+                                       0.f, 0, out_rot, out_rot_interleaved, out_scale, err_flag, dtype, stream);
+}
+
+extern "C" int pg_attention_ragged_tc_capped(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,
+                                             int gate_per_head, const void* k_pool, int ld_k, const void* v_pool, int ld_v,
+                                             long long pool_rows, const int32_t* page_table, int pt_stride, int page_size,
+                                             const int32_t* tiles, int n_tiles, int n_tokens, int n_heads, int n_kv_heads,
+                                             int dim, int vdim, float scale, int window, int keep_first, int chunk,
+                                             const float* slopes, int sigmoid_weights, const float* head_bias,
+                                             const float* sink, float softcap, float temp_coef, int temp_every,
+                                             const float* out_rot, int out_rot_interleaved, float out_scale, int* err_flag,
+                                             int dtype, void* stream) {
   if (n_tiles <= 0) return PG_OK;
   PG_REQUIRE(chunk >= 0 && (chunk == 0 || keep_first == 0), "attention_ragged_tc: blocks of %d positions with %d kept first ones",
              chunk, keep_first);
@@ -347,35 +388,39 @@ extern "C" int pg_attention_ragged_tc_masked(void* out, int ld_out, const void* 
   if (ld_v <= 0) ld_v = n_kv_heads * vdim;
   PG_REQUIRE(ld_k >= n_kv_heads * dim && ld_v >= n_kv_heads * vdim && ld_k % 8 == 0 && ld_v % 8 == 0,
              "attention_ragged_tc: pool rows of %d / %d elements", ld_k, ld_v);
-  PG_REQUIRE(pg_attention_ragged_tc_ok(dim, vdim, page_size, ld_q, ld_out, (gate && !gate_per_head) ? ld_gate : 8, dtype),
+  PG_REQUIRE(pg_attention_ragged_tc_ok8(dim, vdim, page_size, ld_q, ld_out, (gate && !gate_per_head) ? ld_gate : 8, dtype),
              "attention_ragged_tc: unsupported problem (dim %d vdim %d page %d dtype %d)", dim, vdim, page_size, dtype);
+  PG_REQUIRE(!out_rot || vdim % 64 == 0, "attention_ragged_tc: values of %d columns that are turned back", vdim);
+  PG_REQUIRE(softcap >= 0.f && temp_every >= 0 && (temp_every == 0 || softcap > 0.f),
+             "attention_ragged_tc: softcap %g, temperature steps of %d (a temperature needs a cap here)", (double)softcap, temp_every);
   PG_REQUIRE(n_heads % n_kv_heads == 0, "attention_ragged_tc: heads %d / kv heads %d", n_heads, n_kv_heads);
   PG_REQUIRE(((uintptr_t)q % 16) == 0 && ((uintptr_t)out % 16) == 0 && (gate_per_head || ((uintptr_t)gate % 16) == 0) &&
                  ((uintptr_t)k_pool % 16) == 0 && ((uintptr_t)v_pool % 16) == 0,
              "attention_ragged_tc: operands must be 16-byte aligned");
   const bool bf = dtype == PG_BF16;
   CUtensorMap mq, mk, mv;
-  PG_REQUIRE(tc::make_map_2d(&mq, q, n_tokens, (long long)n_heads * dim, ld_q, tc::WQ, bf) &&
-                 tc::make_map_2d(&mk, k_pool, pool_rows, (long long)n_kv_heads * dim, (long long)ld_k, tc::WK, bf) &&
-                 tc::make_map_2d(&mv, v_pool, pool_rows, (long long)n_kv_heads * vdim, (long long)ld_v, tc::WK, bf),
+  PG_REQUIRE(tc::make_map_heads(&mq, q, n_tokens, n_heads, dim, ld_q, tc::WQ, bf) &&
+                 tc::make_map_heads(&mk, k_pool, pool_rows, n_kv_heads, dim, ld_k, tc::WK, bf) &&
+                 tc::make_map_heads(&mv, v_pool, pool_rows, n_kv_heads, vdim, ld_v, tc::WK, bf),
              "attention_ragged_tc: cuTensorMapEncodeTiled failed");
+  const int tied = (k_pool == v_pool && ld_k == ld_v && (dim == vdim || (n_kv_heads == 1 && vdim < dim))) ? 1 : 0;
+  const int bounded = (bf && softcap > 0.f && softcap <= 40.f && !sigmoid_weights && !slopes && !head_bias) ? 1 : 0;
   tc::WinParams p = {out, ld_out, gate, ld_gate, tiles, page_table, pt_stride, n_heads, n_heads / n_kv_heads, dim, vdim,
                      scale, window, slopes, err_flag, keep_first, sigmoid_weights ? 1 : 0, head_bias,
-                     gate_per_head ? 1 : 0, out_scale, sink, chunk, out_rot, out_rot_interleaved ? 1 : 0};
-  const size_t smem = 1024 + (size_t)tc::WQ * dim * 2 + 2 * (size_t)tc::WK * dim * 2 + (size_t)tc::WK * vdim * 2 +
+                     gate_per_head ? 1 : 0, out_scale, sink, chunk, out_rot, out_rot_interleaved ? 1 : 0, softcap, temp_coef,
+                     temp_every, tied, bounded};
+  const int kb = cdiv(dim, 64), vb = cdiv(vdim, 64);
+  const size_t smem = 1024 + (size_t)tc::WQ * kb * 128 + 2 * (size_t)tc::WK * kb * 128 + (tied ? 0 : (size_t)tc::WK * vb * 128) +
                       (size_t)tc::WQ * tc::WK * 2 + 72 + 16;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(n_tiles, n_heads);
-  if (bf) {
-    auto kern = tc::attention_window_tc_kernel<bf16>;
+  auto run = [&](auto kern) -> int {
     PG_REQUIRE(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess,
                "attention_ragged_tc: cannot reserve %zu B of shared memory", smem);
     return launch_tc("attention_ragged_tc", kern, grid, dim3(256), smem, 1, false, st, mq, mk, mv, p);
-  }
-  auto kern = tc::attention_window_tc_kernel<f16>;
-  PG_REQUIRE(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess,
-             "attention_ragged_tc: cannot reserve %zu B of shared memory", smem);
-  return launch_tc("attention_ragged_tc", kern, grid, dim3(256), smem, 1, false, st, mq, mk, mv, p);
+  };
+  if (softcap > 0.f) return bf ? run(tc::attention_window_tc_kernel<bf16, true>) : run(tc::attention_window_tc_kernel<f16, true>);
+  return bf ? run(tc::attention_window_tc_kernel<bf16, false>) : run(tc::attention_window_tc_kernel<f16, false>);
 }
 
 extern "C" int pg_attention_ragged_tc_ex(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate,

@@ -5,8 +5,9 @@
 //                   score * scale (not renormalised); optional per-token sigmoid gate of a shared expert
 //   pg_moe_sort     pairs whose expert index is < n_experts are grouped by expert (offsets, source rows, position of
 //                   each pair); larger indices are identity experts and take no part in the GEMMs
+//   pg_moe_table_sort  experts picked by token id from a table: the grouping of every such layer of a model in one launch
 //   pg_moe_gemm     out[pos] = A[row(pos)] W_e^T for the pairs of every expert e, optionally with the SwiGLU pairing
-//                   silu(A Wg^T) * (A Wu^T) of stacked [Wg; Wu] weights
+//                   silu(A Wg^T) * (A Wu^T) of stacked [Wg; Wu] weights, or with max(A W^T, 0)^2
 //   pg_moe_combine  x[t] += sum_k w_k * (k-th expert's output, or the token's own input for an identity expert)
 //                           + gate[t] * shared[t]
 #include "common.cuh"
@@ -221,6 +222,66 @@ __global__ void moe_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restri
   }
 }
 
+// ------------------------------------------------------------------ experts picked by token id: every layer's grouping at once
+// Routing by a table [vocab, top] of expert indices depends on the token ids alone, so the pairs of ALL such layers are
+// grouped before the first layer runs: CTA l handles layer l.  desc[l] = {first entry of the layer's table in `tables`,
+// experts, top, sum of the earlier layers' top, sum of the earlier layers' (experts + 1)}.  Layer l's pair_pos starts at
+// n_tokens * desc[l][3], its offsets at desc[l][4].  An id outside the vocabulary gets no place (-1).
+__global__ void __launch_bounds__(1024)
+moe_table_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restrict__ pair_pos, const int32_t* __restrict__ tables,
+                      const int32_t* __restrict__ desc, const int64_t* __restrict__ ids, int n_tokens, long long vocab,
+                      int max_experts) {
+  extern __shared__ int sm_i[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int32_t* d = desc + 5 * blockIdx.x;
+  const int E = d[1], top = d[2];
+  const int32_t* table = tables + d[0];
+  int32_t* pos = pair_pos + (size_t)n_tokens * d[3];
+  int32_t* off = offsets + d[4];
+  int* count = sm_i;                   // [max_experts]
+  int* cursor = sm_i + max_experts;    // [max_experts]
+  for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
+  __syncthreads();
+  const int lane = threadIdx.x & 31, n_pairs = n_tokens * top;
+  auto expert_of = [&](int i) {
+    if (i >= n_pairs) return -1;
+    const int64_t id = ids[i / top];
+    const int e = (id >= 0 && id < vocab) ? table[id * top + i % top] : -1;
+    return e < E ? e : -1;
+  };
+  // lanes of a warp that fall on one expert are counted by one atomic (a handful of experts, thousands of pairs)
+  for (int i0 = threadIdx.x - lane; i0 < n_pairs; i0 += blockDim.x) {
+    const int e = expert_of(i0 + lane);
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && (__ffs(same) - 1) == lane) atomicAdd(&count[e], __popc(same));
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {              // exclusive prefix over the experts, 32 at a time
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int c = e0 + lane < E ? count[e0 + lane] : 0;
+      int inc = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, inc, o); if (lane >= o) inc += v; }
+      if (e0 + lane < E) { off[e0 + lane] = base + inc - c; cursor[e0 + lane] = base + inc - c; }
+      base += __shfl_sync(0xffffffffu, inc, 31);
+    }
+    if (lane == 0) off[E] = base;
+  }
+  __syncthreads();
+  // the order of the pairs inside a group does not change any result: every output row is computed on its own
+  for (int i0 = threadIdx.x - lane; i0 < n_pairs; i0 += blockDim.x) {
+    const int i = i0 + lane, e = expert_of(i);
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    const int leader = __ffs(same) - 1, rank = __popc(same & ((1u << lane) - 1u));
+    int at = 0;
+    if (e >= 0 && leader == lane) at = atomicAdd(&cursor[e], __popc(same));
+    at = __shfl_sync(0xffffffffu, at, leader);
+    if (i < n_pairs) pos[i] = e >= 0 ? at + rank : -1;
+  }
+}
+
 // ------------------------------------------------------------------ grouped GEMM, fp32 FMA (any dtype)
 // The gated pairings of a stacked [Wg; Wu] product (g, u already rounded to the model dtype):
 //   PG_GLU_SILU    silu(g) * u
@@ -318,7 +379,8 @@ moe_gemm_simt_kernel(T* __restrict__ out, int ldo, const T* __restrict__ A, int 
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
-      float v = rnd<T>(acc[i][j]);
+      float v = act == PG_ACT_RELU2 ? fmaxf(acc[i][j], 0.f) : rnd<T>(acc[i][j]);
+      if (act == PG_ACT_RELU2) v *= v;
       if (DUAL) v = glu_pair<T>(v, rnd<T>(acu[DUAL ? i : 0][j]), act, limit);
       out[(size_t)m * ldo + n] = from_f<T>(v);
     }
@@ -400,12 +462,23 @@ extern "C" int pg_moe_sort(int32_t* offsets, int32_t* sorted_row, int32_t* pair_
                     (cudaStream_t)stream, offsets, sorted_row, pair_pos, topk_idx, n_pairs, top, n_experts);
 }
 
+extern "C" int pg_moe_table_sort(int32_t* offsets, int32_t* pair_pos, const int32_t* tables, const int32_t* desc, int n_layers,
+                                 const int64_t* ids, int n_tokens, long long vocab, int max_experts, void* stream) {
+  if (n_layers <= 0 || n_tokens <= 0) return PG_OK;
+  PG_REQUIRE(offsets && pair_pos && tables && desc && ids && max_experts >= 1 && max_experts <= 4096,
+             "moe_table_sort: %d layers, up to %d experts", n_layers, max_experts);
+  return launch_pdl("moe_table_sort", moe_table_sort_kernel, dim3(n_layers), dim3(n_tokens <= 64 ? 128 : 1024),
+                    sizeof(int) * 2 * (size_t)max_experts, (cudaStream_t)stream, offsets, pair_pos, tables, desc, ids, n_tokens,
+                    vocab, max_experts);
+}
+
 extern "C" int pg_moe_gemm_act(void* out, int ldo, const void* A, int lda, const int32_t* row_map, const void* W,
                                const int32_t* offsets, int n_pairs, int n_experts, int N, int K, int act, float limit,
                                int impl, int* err_flag, int dtype, void* stream) {
   if (n_pairs <= 0) return PG_OK;
-  PG_REQUIRE(act == PG_GLU_NONE || act == PG_GLU_SILU || act == PG_GLU_CLAMPED, "moe_gemm: unknown pairing %d", act);
-  const int swiglu = act != PG_GLU_NONE;
+  PG_REQUIRE(act == PG_GLU_NONE || act == PG_GLU_SILU || act == PG_GLU_CLAMPED || act == PG_ACT_RELU2,
+             "moe_gemm: unknown pairing or activation %d", act);
+  const int swiglu = act == PG_GLU_SILU || act == PG_GLU_CLAMPED;      // two products per output
   cudaStream_t st = (cudaStream_t)stream;
   if (impl != 1 && moe_gemm_tc_supported(ldo, lda, row_map, N, K, dtype))
     return moe_gemm_tc(out, ldo, A, lda, row_map, W, offsets, n_pairs, n_experts, N, K, act, limit, dtype, err_flag, st);

@@ -24,7 +24,7 @@ struct MoeParams {
   const int32_t* offsets;
   int n_experts, N, K, ldo;
   int* err_flag;   // device-visible int, set to 2 when a pipeline wait gave up (may be NULL)
-  int act;         // pairing of the two products of a stacked [Wg; Wu] tile: PG_GLU_SILU or PG_GLU_CLAMPED
+  int act;         // pairing of the two products of a stacked [Wg; Wu] tile: PG_GLU_SILU or PG_GLU_CLAMPED; of one: PG_ACT_RELU2
   float limit;     // PG_GLU_CLAMPED: g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(1.702 g') (u' + 1)
   // Per-head mode (group_rows > 0; offsets unused): every group is one head of the SAME group_rows token rows.  Group e
   // reads its operand at columns e * a_gs of the token rows (the A map covers the token-major matrix) and writes
@@ -201,7 +201,9 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
             float o[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-              float x = rnd<T>(v[j0 + j]);
+              float x = v[j0 + j];
+              if (!DUAL && p.act == PG_ACT_RELU2) { x = fmaxf(x, 0.f); o[j] = x * x; continue; }
+              x = rnd<T>(x);
               if (DUAL) {
                 float uu = rnd<T>(u[DUAL ? j0 + j : 0]);
                 if (p.act == PG_GLU_CLAMPED) {
@@ -264,7 +266,7 @@ bool moe_gemm_tc_supported(int ldo, int lda, const int32_t* row_map, int N, int 
 int moe_gemm_tc(void* out, int ldo, const void* A, int lda, const int32_t* row_map, const void* W,
                 const int32_t* offsets, int n_pairs, int n_experts, int N, int K, int act, float limit, int dtype,
                 int* err_flag, cudaStream_t st) {
-  const int swiglu = act != PG_GLU_NONE;
+  const int swiglu = act == PG_GLU_SILU || act == PG_GLU_CLAMPED;
   (void)row_map;
   PG_REQUIRE(((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0 && ((uintptr_t)out % 16) == 0,
              "moe_gemm_tc: operands must be 16-byte aligned");

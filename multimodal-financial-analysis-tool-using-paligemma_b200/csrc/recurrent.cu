@@ -21,8 +21,8 @@
 //                                         the current ones are consumed.  The state is loaded from / stored to the
 //                                         slot's state once per launch, which makes a prompt portion and a single
 //                                         decoded token the same case.
-// headnorm_gate_kernel (warp per (token, head)): o / rms(o) per head, times a weight, times sigmoid(gate), times a
-//                                         constant, rounded to the model dtype as the output projection's operand.
+// headnorm_gate_kernel (warp per (token, head)): o / rms(o) per head, times a weight (may be absent), times sigmoid(gate)
+//                                         or silu(gate), times a constant, rounded to the model dtype as the output projection's operand.
 #include "common.cuh"
 
 namespace pg {
@@ -219,7 +219,7 @@ delta_rule_kernel(float* __restrict__ out, float* __restrict__ state, const floa
 template <typename T>
 __global__ void headnorm_gate_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ o, const T* __restrict__ w,
                                      const T* __restrict__ gate, int ld_gate, int n_tokens, int heads, int dim, float eps,
-                                     float out_scale, int pairs) {
+                                     float out_scale, int pairs, int gate_silu) {
   pdl_launch_dependents();
   pdl_wait();
   const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -227,6 +227,7 @@ __global__ void headnorm_gate_kernel(T* __restrict__ out, int ld_out, const floa
   if (item >= (long long)n_tokens * heads) return;
   const int t = (int)(item / heads), h = (int)(item % heads);
   const float* orow = o + ((size_t)t * heads + h) * dim;
+  auto gate_f = [&](float z) { return gate_silu ? z * sigmoid_f(z) : sigmoid_f(z); };
   float ss = 0.f;
   if (pairs) {                                     // two columns per lane and access (even sizes, aligned rows)
     for (int c = 2 * lane; c < dim; c += 64) { const float2 v = *reinterpret_cast<const float2*>(orow + c); ss += v.x * v.x + v.y * v.y; }
@@ -238,7 +239,7 @@ __global__ void headnorm_gate_kernel(T* __restrict__ out, int ld_out, const floa
       if (w) { a *= to_f<T>(w[h * dim + c]); b *= to_f<T>(w[h * dim + c + 1]); }
       if (gate) {
         const T* gp = gate + (size_t)t * ld_gate + h * dim + c;
-        a *= sigmoid_f(to_f<T>(gp[0])); b *= sigmoid_f(to_f<T>(gp[1]));
+        a *= gate_f(to_f<T>(gp[0])); b *= gate_f(to_f<T>(gp[1]));
       }
       T* op = out + (size_t)t * ld_out + h * dim + c;
       if constexpr (sizeof(T) == 2) {
@@ -256,7 +257,7 @@ __global__ void headnorm_gate_kernel(T* __restrict__ out, int ld_out, const floa
   for (int c = lane; c < dim; c += 32) {
     float v = orow[c] * inv;
     if (w) v *= to_f<T>(w[h * dim + c]);
-    if (gate) v *= sigmoid_f(to_f<T>(gate[(size_t)t * ld_gate + h * dim + c]));
+    if (gate) v *= gate_f(to_f<T>(gate[(size_t)t * ld_gate + h * dim + c]));
     out[(size_t)t * ld_out + h * dim + c] = from_f<T>(v * out_scale);
   }
 }
@@ -297,6 +298,96 @@ __global__ void lightning_prep_kernel(float* __restrict__ rec, const T* __restri
       a = a * sigmoid_f(a);
     }
     out[i] = a;
+  }
+}
+
+// Retention (linear attention with rotary positions in place of activations) runs on the same recurrence: its records
+// are written by retention_prep_kernel below.  The first rot_dims columns of every q and k head are turned in pairs
+// (i, i + rot_dims / 2), or (2i, 2i + 1) when interleaved, by position * freq[i]; k is multiplied by k_scale after the
+// rotation; v passes.  freq holds (high, low) float pairs: the angle's rounding error and the low part enter as a first-
+// order correction, so that far positions keep full fp32 accuracy.  One CTA per token: the token's sines and cosines
+// once into shared memory (the heads share them), then records four columns at a time.
+template <typename T>
+__global__ void retention_prep_kernel(float* __restrict__ rec, const T* __restrict__ proj, int ld, int q_col0, int k_col0,
+                                      int v_col0, const float2* __restrict__ freq, int rot_dims, int interleaved, float k_scale,
+                                      const int32_t* __restrict__ tok_pos, int heads, int dim, int vdim, int dp, int vp) {
+  extern __shared__ float2 cs[];                    // [rot_dims / 2] (cos, sin)
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int half = rot_dims >> 1, rs = 2 * dp + vp, rs4 = rs / 4;
+  const float p = (float)tok_pos[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float2 f = freq[i];
+    const float a = p * f.x, d = fmaf(p, f.x, -a) + p * f.y;   // the exact angle is a + d
+    float s, c;
+    sincosf(a, &s, &c);
+    cs[i] = make_float2(c - s * d, s + c * d);
+  }
+  __syncthreads();
+  const T* row = proj + t * ld;
+  float* out = rec + t * heads * rs;
+  auto rotated = [&](const T* head, int c) -> float {          // column c of a q or k head
+    const float u = to_f<T>(head[c]);
+    if (c >= rot_dims) return u;
+    const bool first = interleaved ? !(c & 1) : c < half;
+    const int pair = interleaved ? c >> 1 : (first ? c : c - half);
+    const float w = to_f<T>(head[interleaved ? c ^ 1 : (first ? c + half : c - half)]);
+    const float2 e = cs[pair];
+    return first ? u * e.x - w * e.y : u * e.x + w * e.y;
+  };
+  // pairs of halves with everything in whole groups of four: 8- or 16-byte loads
+  const bool quad = !interleaved && half % 4 == 0 && dim % 4 == 0 && vdim % 4 == 0 && ld % 4 == 0 && q_col0 % 4 == 0 &&
+                    k_col0 % 4 == 0 && v_col0 % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  auto ld4 = [&](const T* q, float* f) {
+    if constexpr (sizeof(T) == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(q);
+      f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+    } else {
+      const uint2 v = *reinterpret_cast<const uint2*>(q);
+      const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) f[k] = to_f<T>(e[k]);
+    }
+  };
+  for (int i = threadIdx.x; i < heads * rs4; i += blockDim.x) {
+    const int h = i / rs4, c0 = (i - h * rs4) * 4;
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+    if (c0 >= 2 * dp) {
+      const int c = c0 - 2 * dp;
+      const T* head = row + v_col0 + h * vdim;
+      if (quad) { ld4(head + c, o); }
+      else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) if (c + k < vdim) o[k] = to_f<T>(head[c + k]);
+      }
+    } else {
+      const bool is_k = c0 >= dp;
+      const int c = is_k ? c0 - dp : c0;
+      const T* head = row + (is_k ? k_col0 : q_col0) + h * dim;
+      const float sc = is_k ? k_scale : 1.f;
+      if (quad) {
+        float u[4];
+        ld4(head + c, u);
+        if (c < rot_dims) {
+          const bool first = c < half;
+          const int pair = first ? c : c - half;
+          float w[4];
+          ld4(head + (first ? c + half : c - half), w);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 e = cs[pair + k];
+            u[k] = first ? u[k] * e.x - w[k] * e.y : u[k] * e.x + w[k] * e.y;
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) o[k] = u[k] * sc;
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) if (c + k < dim) o[k] = rotated(head, c + k) * sc;
+      }
+    }
+    *reinterpret_cast<float4*>(out + (size_t)h * rs + c0) = make_float4(o[0], o[1], o[2], o[3]);
   }
 }
 
@@ -465,6 +556,12 @@ extern "C" int pg_delta_rule(float* out, float* state, const float* rec, const i
 
 extern "C" int pg_headnorm_gate(void* out, int ld_out, const float* o, const void* w, const void* gate, int ld_gate,
                                 int n_tokens, int heads, int dim, float eps, float out_scale, int dtype, void* stream) {
+  return pg_headnorm_gate_ex(out, ld_out, o, w, gate, ld_gate, 0, n_tokens, heads, dim, eps, out_scale, dtype, stream);
+}
+
+extern "C" int pg_headnorm_gate_ex(void* out, int ld_out, const float* o, const void* w, const void* gate, int ld_gate,
+                                   int gate_silu, int n_tokens, int heads, int dim, float eps, float out_scale, int dtype,
+                                   void* stream) {
   if (n_tokens <= 0) return PG_OK;
   PG_REQUIRE(out && o && heads > 0 && dim > 0, "headnorm_gate: bad arguments");
   const int warps = 8;
@@ -473,7 +570,7 @@ extern "C" int pg_headnorm_gate(void* out, int ld_out, const float* o, const voi
   PG_DISPATCH_DTYPE(dtype, T, {
     return launch_pdl("headnorm_gate", headnorm_gate_kernel<T>, dim3(cdiv((long long)n_tokens * heads, warps)),
                       dim3(warps * 32), 0, (cudaStream_t)stream, (T*)out, ld_out, o, (const T*)w, (const T*)gate, ld_gate,
-                      n_tokens, heads, dim, eps, out_scale, pairs);
+                      n_tokens, heads, dim, eps, out_scale, pairs, gate_silu ? 1 : 0);
   });
   return PG_OK;
 }
@@ -490,6 +587,23 @@ extern "C" int pg_lightning_prep(float* rec, const void* proj, int ld, int q_col
   PG_DISPATCH_DTYPE(dtype, T, {
     return launch_pdl("lightning_prep", lightning_prep_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, rec,
                       (const T*)proj, ld, q_col0, k_col0, v_col0, (long long)n_tokens, heads, dim, vdim, dp, vp);
+  });
+  return PG_OK;
+}
+
+extern "C" int pg_retention_prep(float* rec, const void* proj, int ld, int q_col0, int k_col0, int v_col0, const float* freq,
+                                 int rot_dims, int interleaved, float k_scale, const int32_t* tok_pos, int n_tokens, int heads,
+                                 int dim, int vdim, int dtype, void* stream) {
+  if (n_tokens <= 0) return PG_OK;
+  PG_REQUIRE(rec && proj && tok_pos && heads > 0 && dim > 0 && vdim > 0, "retention_prep: bad arguments");
+  PG_REQUIRE(rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && (rot_dims == 0 || freq),
+             "retention_prep: %d rotated columns of %d (even, with a frequency table)", rot_dims, dim);
+  const int dp = (dim + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4;
+  const int work = heads * (2 * dp + vp) / 4, threads = work >= 512 ? 256 : (work >= 128 ? 128 : 64);
+  PG_DISPATCH_DTYPE(dtype, T, {
+    return launch_pdl("retention_prep", retention_prep_kernel<T>, dim3(n_tokens), dim3(threads), sizeof(float) * (size_t)rot_dims,
+                      (cudaStream_t)stream, rec, (const T*)proj, ld, q_col0, k_col0, v_col0, (const float2*)freq, rot_dims,
+                      interleaved ? 1 : 0, k_scale, tok_pos, heads, dim, vdim, dp, vp);
   });
   return PG_OK;
 }

@@ -39,6 +39,12 @@ __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map
       ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(c0), "r"(c1)
       : "memory");
 }
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int c0, int c1, int c2) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+      ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(c0), "r"(c1), "r"(c2)
+      : "memory");
+}
 // The same load delivered to every CTA of the cluster named in cta_mask (same shared-memory offset, same mbarrier offset).
 __device__ __forceinline__ void tma_load_2d_mcast(uint32_t dst, const CUtensorMap* map, uint32_t bar, int c0, int c1,
                                                   uint16_t cta_mask) {
@@ -113,6 +119,10 @@ bool make_map_2d(CUtensorMap* map, const void* base, long long rows, long long c
 // same with an explicit box width (elements) and swizzle span (32 / 64 / 128 bytes; box_cols * 2 <= swizzle_bytes)
 bool make_map_2d_ex(CUtensorMap* map, const void* base, long long rows, long long cols, long long ld, int box_cols,
                     int box_rows, int swizzle_bytes, bool is_bf16);
+// Rows that hold `heads` equal parts of `cols` columns (cols % 8 == 0), as a 3-D tensor {column, head, row}: box = 64 columns
+// of ONE head x box_rows rows, 128-byte swizzle.  Columns behind a head's last one read as zero, not as the next head.
+bool make_map_heads(CUtensorMap* map, const void* base, long long rows, int heads, int cols, long long ld, int box_rows,
+                    bool is_bf16);
 
 }  // namespace tc
 }  // namespace pg

@@ -14,7 +14,8 @@ LIB_PATH = os.environ.get("PG_LIB_PATH") or os.path.join(_HERE, "libpg_b200.so")
 
 PG_F32, PG_BF16, PG_F16 = 0, 1, 2
 EPI_NONE, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RES, EPI_RES, EPI_GEGLU, EPI_SWIGLU = 0, 1, 2, 3, 4, 5, 6
-GLU_NONE, GLU_SILU, GLU_CLAMPED = 0, 1, 2      # pairings of pg_moe_gemm_act
+GLU_NONE, GLU_SILU, GLU_CLAMPED, ACT_RELU2 = 0, 1, 2, 3      # pairings / activation of pg_moe_gemm_act
+EMB_NONE, EMB_INIT, EMB_ADD = 0, 1, 2          # what pg_residual_layernorm does with the embedding row
 MAX_DECODE_BATCH = 8            # rows one launch of the GEMV kernels can take
 # from this batch size on the decode step runs the tensor-core (swap-AB skinny GEMM) path: the GEMV kernels turn
 # ALU-bound as rows are added (batch 8: 4.34 ms/step vs ~2 ms), tools/kernel_sweep.py SWEEP_B=...
@@ -124,6 +125,18 @@ SIGNATURES = {
     "pg_ssm_prep": [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "pg_gate_groupnorm": [_vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _f, _i, _vp],
     "pg_lightning_attention_ex": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    # layer norms between sublayers, experts picked by token id, retention, capped attention over tied values
+    "pg_residual_layernorm": [_vp, _i, _vp, _vp, _i, _vp, _i, _f, _vp, _vp, _ll, _i, _vp, _vp, _vp, _f, _f, _vp, _vp, _i, _i,
+                              _i, _vp, _i, _vp],
+    "pg_cache_append": [_vp, _i, _vp, _i, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _vp],
+    "pg_moe_table_sort": [_vp, _vp, _vp, _vp, _i, _vp, _i, _ll, _i, _vp],
+    "pg_retention_prep": [_vp, _vp, _i, _i, _i, _i, _vp, _i, _i, _f, _vp, _i, _i, _i, _i, _i, _vp],
+    "pg_headnorm_gate_ex": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
+    "pg_attention_ragged_capped": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i,
+                                   _i, _f, _i, _i, _i, _vp, _i, _vp, _vp, _f, _f, _i, _vp, _i, _f, _vp, _ll, _i, _vp],
+    "pg_attention_ragged_tc_ok8": [_i, _i, _i, _i, _i, _i, _i],
+    "pg_attention_ragged_tc_capped": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _ll, _vp, _i, _i, _vp, _i, _i, _i, _i,
+                                      _i, _i, _f, _i, _i, _i, _vp, _i, _vp, _vp, _f, _f, _i, _vp, _i, _f, _vp, _i, _vp],
 }
 _RESTYPE = {"pg_last_error": C.c_char_p, "pg_launch_count": _ull, "pg_decode_attention_ws_floats": _ll,
             "pg_delta_record_floats": _ll, "pg_lightning_record_floats": _ll, "pg_ssm_record_floats": _ll}

@@ -47,7 +47,7 @@ import torch
 from . import _cabi as cabi
 from ._cabi import ptr
 from .latent import LatentAttentionMixin, LatentCfg, latent_cfg, pack_latent
-from .ragged_engine import RaggedEngine, StepInputs, _stack_rows
+from .ragged_engine import LoopCfg, RaggedEngine, Run, StepInputs, _stack_rows, layer_runs, loop_cfg
 from .registry import register
 
 GLU_ALPHA = 1.702                 # the sigmoid's slope in the experts' activation: fixed by the design
@@ -81,19 +81,6 @@ class LayerCfg:
 
 
 @dataclass
-class LoopCfg:
-    start: int
-    stop: int
-    times: int
-
-
-@dataclass
-class Run:
-    layer: int
-    loop_pass: Optional[int]      # the number of the pass this run opens (its first layer), else None
-
-
-@dataclass
 class BirizenConfig:
     vocab: int
     width: int
@@ -103,14 +90,7 @@ class BirizenConfig:
 
     def runs(self) -> List[Run]:
         """The layer runs of one forward pass, in order."""
-        n = len(self.layers)
-        if self.loop is None:
-            return [Run(i, None) for i in range(n)]
-        lp = self.loop
-        out = [Run(i, None) for i in range(lp.start)]
-        for t in range(lp.times):
-            out += [Run(i, t if i == lp.start else None) for i in range(lp.start, lp.stop)]
-        return out + [Run(i, None) for i in range(lp.stop, n)]
+        return layer_runs(len(self.layers), self.loop)
 
     @staticmethod
     def from_dict(cfg: Mapping) -> "BirizenConfig":
@@ -142,12 +122,7 @@ class BirizenConfig:
                     raise ValueError(f"layer {i}: top {mlp.top} of {mlp.experts} experts in {mlp.groups} groups, "
                                      f"{mlp.keep} kept")
             layers.append(LayerCfg(kind, mixer, mlp))
-        lp = cfg.get("loop")
-        loop = None
-        if lp:
-            loop = LoopCfg(int(lp["start"]), int(lp["stop"]), int(lp["times"]))
-            if not (0 <= loop.start < loop.stop <= len(layers)) or loop.times < 1:
-                raise ValueError(f"loop over layers {loop.start} .. {loop.stop - 1}, {loop.times} times")
+        loop = loop_cfg(cfg.get("loop"), len(layers))
         return BirizenConfig(vocab=int(cfg["vocab"]), width=int(cfg["width"]), eps=float((cfg.get("norm") or {})["eps"]),
                              layers=layers, loop=loop)
 

@@ -77,6 +77,40 @@ class RotaryCfg:
 
 
 
+@dataclass
+class LoopCfg:
+    """Layers start .. stop-1 run `times` times in a row with the same weights (every pass has its own cache / state)."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
+class Run:
+    layer: int
+    loop_pass: Optional[int]      # the number of the pass this run opens (its first layer), else None
+
+
+def loop_cfg(entry, n_layers: int) -> Optional[LoopCfg]:
+    """The looped block from a config's `loop` entry (absent or empty: none)."""
+    if not entry:
+        return None
+    loop = LoopCfg(int(entry["start"]), int(entry["stop"]), int(entry["times"]))
+    if not (0 <= loop.start < loop.stop <= n_layers) or loop.times < 1:
+        raise ValueError(f"loop over layers {loop.start} .. {loop.stop - 1}, {loop.times} times")
+    return loop
+
+
+def layer_runs(n_layers: int, loop: Optional[LoopCfg]) -> List[Run]:
+    """The layer runs of one forward pass, in order."""
+    if loop is None:
+        return [Run(i, None) for i in range(n_layers)]
+    out = [Run(i, None) for i in range(loop.start)]
+    for t in range(loop.times):
+        out += [Run(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
+    return out + [Run(i, None) for i in range(loop.stop, n_layers)]
+
+
 def _stack_rows(parts, device, dtype, align=8):
     """Concatenate [rows_i, K] matrices with every part starting at a multiple of `align` rows (zero rows between),
     so that the columns of the fused projection's output start aligned.  Returns (matrix, {name: first row})."""
@@ -190,22 +224,34 @@ class RaggedEngine(PagePool):
         rows, pos = self._new(P, dtype=torch.int32), self._new(P, dtype=torch.int32)
         with tm("moe_sort"):
             cabi.check(L.pg_moe_sort(ptr(offsets), ptr(rows), ptr(pos), ptr(idx), P, top, E, st), "moe_sort")
-        act_out, y = self._new(P, ff), self._new(P, D)
-        tc = (self.dtype != torch.float32 and self.moe_impl != 1 and P >= self.moe_tc_min_pairs
-              and D % 8 == 0 and ff % 8 == 0)
-        a, row_map, impl = h, rows, 1
-        if tc:
-            a, row_map, impl = self._new(P, D), None, 2
+        a, row_map = h, rows
+        if self._moe_tc(P, D, ff):
+            a, row_map = self._new(P, D), None
             with tm("moe_gather"):
                 cabi.check(L.pg_gather_rows(ptr(a), ptr(h), h.stride(0), ptr(rows), ptr(offsets[E:]), P, D, self.dt, st),
                            "gather_rows")
-        with tm("moe_gate_up"):
+        return self._moe_ffn(a, row_map, offsets, P, E, ff, w_gu, w_dn, act, limit), pos
+
+    def _moe_tc(self, pairs: int, D: int, ff: int) -> bool:
+        """Whether the grouped expert GEMMs of this step run on the tensor cores."""
+        return (self.dtype != torch.float32 and self.moe_impl != 1 and pairs >= self.moe_tc_min_pairs
+                and D % 8 == 0 and ff % 8 == 0)
+
+    def _moe_ffn(self, a: torch.Tensor, row_map, offsets, P: int, E: int, ff: int, w_gu: torch.Tensor, w_dn: torch.Tensor,
+                 act: int, limit: float = 0.0) -> torch.Tensor:
+        """Both grouped expert GEMMs over P pairs in expert order: y [P, D].  a holds the rows in that order (row_map
+        None), or the rows that row_map picks (fp32-FMA kernel only).  w_gu is [E, 2 ff, D] for a gated pairing,
+        [E, ff, D] for an activation of one product; w_dn [E, D, ff]."""
+        L, st, tm, D = cabi.lib(), cabi.stream(), self._tm, a.shape[1]
+        impl = 2 if row_map is None and self._moe_tc(P, D, ff) else 1
+        act_out, y = self._new(P, ff), self._new(P, D)
+        with tm("moe_gate_up" if act in (cabi.GLU_SILU, cabi.GLU_CLAMPED) else "moe_up"):
             cabi.check(L.pg_moe_gemm_act(ptr(act_out), ff, ptr(a), a.stride(0), ptr(row_map), ptr(w_gu), ptr(offsets), P, E,
-                                         ff, D, act, limit, impl, ptr(self.err_flag), self.dt, st), "moe_gemm gate/up")
+                                         ff, D, act, limit, impl, ptr(self.err_flag), self.dt, st), "moe_gemm up")
         with tm("moe_down"):
             cabi.check(L.pg_moe_gemm_act(ptr(y), D, ptr(act_out), ff, None, ptr(w_dn), ptr(offsets), P, E, D, ff,
                                          cabi.GLU_NONE, 0.0, impl, ptr(self.err_flag), self.dt, st), "moe_gemm down")
-        return y, pos
+        return y
 
     # ------------------------------------------------------------------ one step
     @staticmethod

@@ -37,6 +37,7 @@ def _load_builtin() -> None:
     from . import gogivik  # noqa: F401
     from . import mubasun  # noqa: F401
     from . import ninisun  # noqa: F401
+    from . import ranesun  # noqa: F401
     from . import engine   # noqa: F401
 
 
