@@ -324,7 +324,10 @@ class RaggedEngine(PagePool):
         """Small steps are launch-bound (some fifteen launches per layer): the kernel sequence for (T tokens, nw
         wanted rows) over this slot table is captured once; a step copies its ids / slots / positions into the
         graph's static input and replays.  Which kernels run depends on the counts only, never on the values."""
-        key = (T, nw, ns, kv.page_table.data_ptr(), kv.max_pages)
+        # the captured launches hold the addresses of the page table and of the sequences' state: another slot table may
+        # get the one at an old address and the other at a new one
+        state = () if kv.state is None else tuple(t.data_ptr() for t in kv.state.layers.values())
+        key = (T, nw, ns, kv.page_table.data_ptr(), kv.max_pages, state)
         ent = self._graphs.get(key)
         if ent is None:
             static_in = torch.zeros(host.numel(), dtype=torch.int32, device=self.device)
