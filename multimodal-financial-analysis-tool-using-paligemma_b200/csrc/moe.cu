@@ -227,6 +227,8 @@ __global__ void moe_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restri
 // grouped before the first layer runs: CTA l handles layer l.  desc[l] = {first entry of the layer's table in `tables`,
 // experts, top, sum of the earlier layers' top, sum of the earlier layers' (experts + 1)}.  Layer l's pair_pos starts at
 // n_tokens * desc[l][3], its offsets at desc[l][4].  An id outside the vocabulary gets no place (-1).
+constexpr int SORT_ITEMS = 16;
+
 __global__ void __launch_bounds__(1024)
 moe_table_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restrict__ pair_pos, const int32_t* __restrict__ tables,
                       const int32_t* __restrict__ desc, const int64_t* __restrict__ ids, int n_tokens, long long vocab,
@@ -243,18 +245,27 @@ moe_table_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restrict__ pair_
   int* cursor = sm_i + max_experts;    // [max_experts]
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  const int lane = threadIdx.x & 31, n_pairs = n_tokens * top;
-  auto expert_of = [&](int i) {
-    if (i >= n_pairs) return -1;
-    const int64_t id = ids[i / top];
-    const int e = (id >= 0 && id < vocab) ? table[id * top + i % top] : -1;
-    return e < E ? e : -1;
+  const int lane = threadIdx.x & 31, n_pairs = n_tokens * top, round = SORT_ITEMS * blockDim.x;
+  int ex[SORT_ITEMS];                  // a round's experts of this thread: all its loads are in flight together
+  auto load_round = [&](int i0) {
+    int64_t id[SORT_ITEMS];
+#pragma unroll
+    for (int k = 0; k < SORT_ITEMS; ++k) {
+      const int i = i0 + k * blockDim.x + threadIdx.x;
+      id[k] = i < n_pairs ? ids[i / top] : -1;
+    }
+#pragma unroll
+    for (int k = 0; k < SORT_ITEMS; ++k) {
+      const int i = i0 + k * blockDim.x + threadIdx.x;
+      const int e = (id[k] >= 0 && id[k] < vocab) ? table[id[k] * top + i % top] : -1;
+      ex[k] = e < E ? e : -1;
+    }
   };
-  // lanes of a warp that fall on one expert are counted by one atomic (a handful of experts, thousands of pairs)
-  for (int i0 = threadIdx.x - lane; i0 < n_pairs; i0 += blockDim.x) {
-    const int e = expert_of(i0 + lane);
-    const unsigned same = __match_any_sync(0xffffffffu, e);
-    if (e >= 0 && (__ffs(same) - 1) == lane) atomicAdd(&count[e], __popc(same));
+  for (int i0 = 0; i0 < n_pairs; i0 += round) {
+    load_round(i0);
+#pragma unroll
+    for (int k = 0; k < SORT_ITEMS; ++k)
+      if (ex[k] >= 0) atomicAdd(&count[ex[k]], 1);
   }
   __syncthreads();
   if (threadIdx.x < 32) {              // exclusive prefix over the experts, 32 at a time
@@ -271,14 +282,13 @@ moe_table_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restrict__ pair_
   }
   __syncthreads();
   // the order of the pairs inside a group does not change any result: every output row is computed on its own
-  for (int i0 = threadIdx.x - lane; i0 < n_pairs; i0 += blockDim.x) {
-    const int i = i0 + lane, e = expert_of(i);
-    const unsigned same = __match_any_sync(0xffffffffu, e);
-    const int leader = __ffs(same) - 1, rank = __popc(same & ((1u << lane) - 1u));
-    int at = 0;
-    if (e >= 0 && leader == lane) at = atomicAdd(&cursor[e], __popc(same));
-    at = __shfl_sync(0xffffffffu, at, leader);
-    if (i < n_pairs) pos[i] = e >= 0 ? at + rank : -1;
+  for (int i0 = 0; i0 < n_pairs; i0 += round) {
+    if (n_pairs > round) load_round(i0);            // a single round is still in registers
+#pragma unroll
+    for (int k = 0; k < SORT_ITEMS; ++k) {
+      const int i = i0 + k * blockDim.x + threadIdx.x;
+      if (i < n_pairs) pos[i] = ex[k] >= 0 ? atomicAdd(&cursor[ex[k]], 1) : -1;
+    }
   }
 }
 

@@ -8,6 +8,10 @@ way, a dense Mubasun of equal width, depth, head layout, window and feed-forward
 a mask, dense feed-forward, a recurrence with a gated norm) and Birizen (latent attention with a sink, the decayed
 linear-attention scan the state-space layer runs on) (`run_gogivik`).
 
+`bench.py --arch ranesun`: the Ranesun engine beside the models that hold its closest kernels: the MoE Mubasun (attention,
+norms, experts), Birizen (the decayed linear-attention scan) and Ninisun (the GeGLU feed-forward, the gated head norm)
+(`run_ranesun`).
+
 Timing: CUDA events on the launching stream, >= 3 warm-up steps, an L2-sized scratch write between timed steps.
 Roofline of an op = max(algorithmic FLOPs / measured bf16 peak, algorithmic bytes / measured copy bandwidth);
 `frac` = that time / measured time (1.0 = on the roofline)."""
@@ -605,7 +609,7 @@ def random_birizen_weights(cfg: dict, device, dtype, seed=0) -> Dict[str, torch.
     return out
 
 
-def _birizen_run_layers(s: dict, cfg: dict) -> List[dict]:
+def _looped_layers(s: dict, cfg: dict) -> List[dict]:
     a, b, times = s["loop"]
     order = list(range(a)) + list(range(a, b)) * times + list(range(b, s["layers"]))
     return [cfg["layers"][i] for i in order]
@@ -627,7 +631,7 @@ def birizen_work(s: dict, cfg: dict, T1: int, seqs: int) -> Dict[str, tuple]:
     all_keys = seqs * T1 * (T1 + 1) // 2
     add("norm", 0, (1 + s["loop"][2]) * T * D * (4 + 4 + 2))
     add("loop_in", s["loop"][2] * 2 * T * 2 * D * D, s["loop"][2] * (T * D * (8 + 4 + 4) + 2 * 2 * D * D))
-    for L in _birizen_run_layers(s, cfg):
+    for L in _looped_layers(s, cfg):
         if L["type"] == "lightning":
             nk, nv = H * dim, H * vdim
             npj = 2 * nk + 2 * nv
@@ -664,7 +668,7 @@ def _birizen_decode_bytes(s: dict, cfg: dict, B: int) -> float:
     """Weight bytes one decode step of B tokens must stream (experts: at most B * top of them per MoE layer run)."""
     D, n = s["width"], 0.0
     H, dim, vdim, rot, qr, kr = s["heads"], s["dim"], s["vdim"], s["rot_dim"], s["q_rank"], s["kv_rank"]
-    for L in _birizen_run_layers(s, cfg):
+    for L in _looped_layers(s, cfg):
         if L["type"] == "lightning":
             n += D * (2 * H * dim + 3 * H * vdim)
         else:
@@ -928,6 +932,192 @@ def run_gogivik(sizes, steps: int, warmup: int, peaks: dict, prefill_tokens=2048
                 if a in row["prefill_ops"] and bname in other["prefill_ops"]:
                     fa, fb = row["prefill_ops"][a]["frac"], other["prefill_ops"][bname]["frac"]
                     cmpr[a] = {"frac": fa, "like": bname, "like_frac": fb, "distance_ratio": round(fb / fa, 2) if fa > 0 else None}
+        row["like_for_like"] = cmpr
+        result[name] = row
+    result["gpu_launches"] = int(cabi.launch_count() - launches0)
+    return result
+
+
+# ---------------------------------------------------------------------------------------------------------------
+RANESUN_SIZES = {
+    # head layout, feed-forward and expert sizes of the Mubasun rows; retention heads as Birizen's lightning heads;
+    # layers 1 and 2 run twice
+    "w1024": dict(width=1024, layers=4, heads=8, kv_heads=2, dim=128, ret_heads=8, ret_dim=128, ret_vdim=128, ff=4096, experts=8,
+                  top=2, expert_ff=1024, loop=(1, 3, 2), vocab=32000),
+    "w2048": dict(width=2048, layers=4, heads=16, kv_heads=4, dim=128, ret_heads=16, ret_dim=128, ret_vdim=128, ff=8192, experts=16,
+                  top=2, expert_ff=2048, loop=(1, 3, 2), vocab=32000),
+}
+
+
+def ranesun_config(s: dict) -> dict:
+    """attention + dense, retention + experts, attention + experts, retention + dense, ... (every branch of the design is on
+    the path)."""
+    layers = []
+    for i in range(s["layers"]):
+        if i % 2 == 0:
+            L = {"type": "attention", "mixer": {
+                "heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"],
+                "scale": 1.0 / math.sqrt(s["dim"]), "softcap": 30.0, "q_temp": {"coef": 0.1, "every": 1024}}}
+        else:
+            H = s["ret_heads"]
+            L = {"type": "retention", "mixer": {
+                "heads": H, "dim": s["ret_dim"], "vdim": s["ret_vdim"], "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * h / H) for h in range(H)],
+                "rot": {"dims": s["ret_dim"], "base": 10000.0}}}
+        L["mlp"] = {"kind": "dense", "ff": s["ff"]} if i % 4 in (0, 3) else {
+            "kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+        layers.append(L)
+    return {"architecture": "Ranesun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers,
+            "logit_scale": 1.0, "loop": dict(zip(("start", "stop", "times"), s["loop"]))}
+
+
+def random_ranesun_weights(cfg: dict, device, dtype, seed=0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(seed)
+    D, out = cfg["width"], {}
+
+    def lin(name, o, i):
+        out[name] = (torch.randn(o, i, generator=g, device=device) / math.sqrt(i)).to(dtype)
+
+    def vec(name, n, mean=0.0, std=0.1):
+        out[name] = (mean + std * torch.randn(n, generator=g, device=device)).to(dtype)
+
+    out["embed"] = torch.randn(cfg["vocab"], D, generator=g, device=device).to(dtype)
+    out["loop.step"] = (0.1 * torch.randn(cfg["loop"]["times"], D, generator=g, device=device)).to(dtype)
+    for i, L in enumerate(cfg["layers"]):
+        p, m, ml = f"l{i}.", L["mixer"], L["mlp"]
+        for n in ("norm1", "norm2"):
+            vec(p + n, D, 1.0), vec(p + n + ".b", D)
+        H, d = m["heads"], m["dim"]
+        lin(p + "mix.q", H * d, D)
+        if L["type"] == "attention":
+            lin(p + "mix.k", m["kv_heads"] * d, D), vec(p + "mix.sink", H, 0.0, 1.0), lin(p + "mix.o", D, H * d)
+        else:
+            lin(p + "mix.k", H * d, D), lin(p + "mix.v", H * m["vdim"], D), lin(p + "mix.g", H * m["vdim"], D)
+            lin(p + "mix.o", D, H * m["vdim"])
+        if ml["kind"] == "dense":
+            lin(p + "mlp.gate", ml["ff"], D), lin(p + "mlp.up", ml["ff"], D), lin(p + "mlp.down", D, ml["ff"])
+        else:
+            E, top = ml["router"]["experts"], ml["router"]["top"]
+            for e in range(E):
+                lin(f"{p}mlp.e{e}.up", ml["expert"]["ff"], D), lin(f"{p}mlp.e{e}.down", D, ml["expert"]["ff"])
+            out[p + "mlp.table"] = torch.rand(cfg["vocab"], E, generator=g, device=device).topk(top, -1).indices.to(torch.int32)
+    vec("final.norm", D, 1.0), vec("final.norm.b", D)
+    return out
+
+
+def ranesun_work(s: dict, cfg: dict, T1: int, seqs: int) -> Dict[str, tuple]:
+    """name -> (FLOPs, bytes) of one step over `seqs` prompts of T1 tokens (bf16 operands, fp32 residual stream, fp32 scan
+    records), summed over the layer runs."""
+    T, D, top = T1 * seqs, s["width"], s["top"]
+    P = T * top
+    w: Dict[str, List[float]] = {}
+
+    def add(name, flops, nbytes):
+        a = w.setdefault(name, [0.0, 0.0])
+        a[0] += flops
+        a[1] += nbytes
+
+    def gemm(name, N, K):
+        add(name, 2 * T * N * K, 2 * (T * K + N * K + T * N))
+
+    all_keys = seqs * T1 * (T1 + 1) // 2
+    prev = None                                          # rows of the sublayer output that the next norm sums in, per token
+    for ri, L in enumerate(_looped_layers(s, cfg)):
+        m, ml = L["mixer"], L["mlp"]
+        add("norm", 0, T * D * ((2 + 4) if prev is None else (4 + 4 + 2 * prev)) + T * D * 2)
+        if L["type"] == "attention":
+            H, G, d = m["heads"], m["kv_heads"], m["dim"]
+            gemm("proj", H * d + G * d, D)
+            add("cache_append", 0, 2 * 2 * T * G * d)
+            add("attention", 2 * all_keys * H * 2 * d, 2 * T * (2 * H * d + G * d))
+            gemm("o", D, H * d)
+        else:
+            H, d, e = m["heads"], m["dim"], m["vdim"]
+            rec = H * (2 * d + e)
+            gemm("proj", 2 * H * d + 2 * H * e, D)
+            add("retention_prep", 0, T * rec * (2 + 4))
+            add("retention", 4 * T * H * d * e, T * 4 * (rec + H * e))               # fp32 FMAs, not tensor work
+            add("headnorm_gate", 0, T * H * e * (4 + 2 + 2))
+            gemm("o", D, H * e)
+        if ml["kind"] == "dense":
+            F = ml["ff"]
+            add("norm", 0, T * D * (4 + 4 + 2 + 2))
+            add("gate_up", 2 * T * D * 2 * F, 2 * (T * D + 2 * F * D + T * F))
+            gemm("down", D, F)
+            prev = 1
+        else:
+            E, F = ml["router"]["experts"], ml["expert"]["ff"]
+            add("norm_scatter", 0, T * D * (4 + 4 + 2 + 2 * top))
+            add("moe_up", 2 * P * D * F, 2 * (P * D + E * F * D + P * F))
+            add("moe_down", 2 * P * F * D, 2 * (P * F + E * F * D + P * D))
+            prev = top
+    n_moe = sum(1 for L in cfg["layers"] if L["mlp"]["kind"] == "moe")
+    add("moe_table_sort", 0, n_moe * (8 * T + 4 * 2 * P))                # ids and table entries in, places out
+    add("head", 2 * seqs * D * s["vocab"], 2 * D * s["vocab"])
+    return {k: (v[0], v[1]) for k, v in w.items()}
+
+
+def _ranesun_decode_bytes(s: dict, cfg: dict, B: int) -> float:
+    """Weight bytes one decode step of B tokens must stream (experts: at most B * top of them per MoE layer run)."""
+    D, n = s["width"], 0.0
+    for L in _looped_layers(s, cfg):
+        m, ml = L["mixer"], L["mlp"]
+        if L["type"] == "attention":
+            n += D * m["dim"] * (2 * m["heads"] + m["kv_heads"])
+        else:
+            n += D * m["heads"] * (2 * m["dim"] + 3 * m["vdim"])
+        n += 3 * D * ml["ff"] if ml["kind"] == "dense" else min(s["experts"], B * s["top"]) * 2 * D * s["expert_ff"]
+    return 2.0 * (n + D * s["vocab"])
+
+
+RANESUN_LIKE_MUBASUN = [("proj", "proj"), ("attention", "attention"), ("o", "o"), ("cache_append", "qknorm_append"),
+                        ("norm", "norm"), ("norm_scatter", "norm"), ("moe_table_sort", "moe_sort"), ("moe_up", "moe_gate_up"),
+                        ("moe_down", "moe_down"), ("head", "head")]
+RANESUN_LIKE_BIRIZEN = [("retention", "lightning"), ("retention_prep", "lightning_prep")]
+RANESUN_LIKE_NINISUN = [("gate_up", "gate_up"), ("down", "down"), ("headnorm_gate", "headnorm_gate")]
+
+
+@torch.no_grad()
+def run_ranesun(sizes, steps: int, warmup: int, peaks: dict, prefill_tokens=2048, prefill_seqs=4, context=1024,
+                decode_batches=(1, 8)) -> dict:
+    from .birizen import BirizenEngine
+    from .mubasun import MubasunEngine
+    from .ninisun import NinisunEngine
+    from .ranesun import RanesunEngine
+    dev, dtype = torch.device("cuda:0"), torch.bfloat16
+    timer = _Timer()
+    result = {}
+    launches0 = cabi.launch_count()
+    pool = (max(max(decode_batches), prefill_seqs) + 1) * (max(prefill_tokens, context) + 256)
+
+    def measure(cls, cfg, weights, size, work, decode_bytes):
+        eng = cls(cfg, weights, device=dev, dtype=dtype, kv_pool_tokens=pool)
+        out = _measure_ragged(eng, size["vocab"], timer, steps, warmup, peaks, work(size, cfg, prefill_tokens, prefill_seqs),
+                              decode_bytes, prefill_tokens, prefill_seqs, context, decode_batches)
+        del eng
+        torch.cuda.empty_cache()
+        return out
+
+    for name in sizes:
+        s, ms_, bs_, ns_ = RANESUN_SIZES[name], SIZES[name], BIRIZEN_SIZES[name], NINISUN_SIZES[name]
+        cfg, mcfg, bcfg, ncfg = ranesun_config(s), mubasun_config(ms_), birizen_config(bs_), ninisun_config(ns_)
+        row = {"size": s}
+        row.update(measure(RanesunEngine, cfg, random_ranesun_weights(cfg, dev, dtype), s, ranesun_work,
+                           lambda B: _ranesun_decode_bytes(s, cfg, B)))
+        row["mubasun_equal_size"] = measure(MubasunEngine, mcfg, random_mubasun_weights(mcfg, dev, dtype), ms_, mubasun_work,
+                                            lambda B: _decode_bytes(ms_, mcfg, B))
+        row["birizen_equal_size"] = measure(BirizenEngine, bcfg, random_birizen_weights(bcfg, dev, dtype), bs_, birizen_work,
+                                            lambda B: _birizen_decode_bytes(bs_, bcfg, B))
+        row["ninisun_equal_size"] = measure(NinisunEngine, ncfg, random_ninisun_weights(ncfg, ns_, dev, dtype), ns_, ninisun_work,
+                                            lambda B: _ninisun_decode_bytes(ns_, ncfg))
+        cmpr = {}
+        for like, other in ((RANESUN_LIKE_MUBASUN, "mubasun_equal_size"), (RANESUN_LIKE_BIRIZEN, "birizen_equal_size"),
+                            (RANESUN_LIKE_NINISUN, "ninisun_equal_size")):
+            ops = row[other]["prefill_ops"]
+            for a, bname in like:
+                if a in row["prefill_ops"] and bname in ops:
+                    fa, fb = row["prefill_ops"][a]["frac"], ops[bname]["frac"]
+                    cmpr[a] = {"frac": fa, "like": f"{bname} ({other.split('_')[0]})", "like_frac": fb,
+                               "distance_ratio": round(fb / fa, 2) if fa > 0 else None}
         row["like_for_like"] = cmpr
         result[name] = row
     result["gpu_launches"] = int(cabi.launch_count() - launches0)
