@@ -264,6 +264,16 @@ __device__ __forceinline__ float gelu_tanh_fast(float x) {
   return 0.5f * x * (1.f + t);
 }
 
+// sin and cos of position * frequency, the frequency given as a (high, low) fp32 pair: the product's rounding error and
+// the low part enter as a first-order correction, so that far positions keep full fp32 accuracy.
+__device__ __forceinline__ void rotary_sincos(float pos, float f_hi, float f_lo, float* sn, float* cs) {
+  const float a = pos * f_hi, d = fmaf(pos, f_hi, -a) + pos * f_lo;   // the exact angle is a + d
+  float s, c;
+  sincosf(a, &s, &c);
+  *sn = s + c * d;
+  *cs = c - s * d;
+}
+
 // Orderable 64-bit key for (value, index) argmax: larger value wins, ties go to the LOWER index
 // (torch.argmax returns the first maximal element).
 __device__ __forceinline__ unsigned long long argmax_key(float v, unsigned idx) {

@@ -24,8 +24,8 @@ namespace pg {
 template <typename T>
 __global__ void latent_prep_kernel(T* __restrict__ cq_out, const T* __restrict__ proj, int ld, int dq_col0, int q_rank,
                                    const T* __restrict__ w_q, int dkv_col0, int kv_rank, const T* __restrict__ w_kv,
-                                   int rot_dim, const float* __restrict__ freq, float mag, float eps,
-                                   T* __restrict__ pool, int ld_pool, const int32_t* __restrict__ page_table,
+                                   int rot_dim, const float* __restrict__ freq, const float* __restrict__ freq_lo, int halves,
+                                   float mag, float eps, T* __restrict__ pool, int ld_pool, const int32_t* __restrict__ page_table,
                                    int pt_stride, int page_size, const int32_t* __restrict__ tok_slot,
                                    const int32_t* __restrict__ tok_pos) {
   __shared__ float red[32];
@@ -50,36 +50,40 @@ __global__ void latent_prep_kernel(T* __restrict__ cq_out, const T* __restrict__
     dst[c] = from_f<T>(to_f<T>(row[dkv_col0 + c]) * inv_kv * to_f<T>(w_kv[c]));
   const float fp = (float)p;
   for (int i = threadIdx.x; i < rot_dim / 2; i += blockDim.x) {
-    const float a = to_f<T>(row[dkv_col0 + kv_rank + 2 * i]), b = to_f<T>(row[dkv_col0 + kv_rank + 2 * i + 1]);
+    const int c0 = kv_rank + (halves ? i : 2 * i), c1 = halves ? c0 + rot_dim / 2 : c0 + 1;
+    const float a = to_f<T>(row[dkv_col0 + c0]), b = to_f<T>(row[dkv_col0 + c1]);
     float sn, cs;
-    sincosf(fp * freq[i], &sn, &cs);
+    rotary_sincos(fp, freq[i], freq_lo ? freq_lo[i] : 0.f, &sn, &cs);
     sn *= mag; cs *= mag;
-    dst[kv_rank + 2 * i] = from_f<T>(a * cs - b * sn);
-    dst[kv_rank + 2 * i + 1] = from_f<T>(b * cs + a * sn);
+    dst[c0] = from_f<T>(a * cs - b * sn);
+    dst[c1] = from_f<T>(b * cs + a * sn);
   }
   for (int c = kv_rank + rot_dim + threadIdx.x; c < ld_pool; c += blockDim.x) dst[c] = from_f<T>(0.f);
 }
 
 // ------------------------------------------------------------------ rotated columns of every head of a row
-// dst[t, h * dst_hs + dst_col0 + (2i, 2i+1)] = rotation of src[t, h * src_hs + src_col0 + (2i, 2i+1)] by pos[t] * freq[i]
+// dst[t, h * dst_hs + dst_col0 + (2i, 2i+1)] = rotation of src[t, h * src_hs + src_col0 + (2i, 2i+1)] by pos[t] * freq[i];
+// halves != 0: the pairs are (i, i + rot_dim / 2) instead
 template <typename T>
 __global__ void rotary_cols_kernel(T* __restrict__ dst, int ld_dst, int dst_col0, int dst_hs, const T* __restrict__ src,
                                    int ld_src, int src_col0, int src_hs, int heads, int rot_dim,
-                                   const float* __restrict__ freq, float mag, const int32_t* __restrict__ tok_pos) {
+                                   const float* __restrict__ freq, const float* __restrict__ freq_lo, int halves, float mag,
+                                   const int32_t* __restrict__ tok_pos) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, half = rot_dim / 2;
   const float fp = (float)tok_pos[t];
   for (int idx = threadIdx.x; idx < heads * half; idx += blockDim.x) {
     const int h = idx / half, i = idx % half;
-    const T* s = src + (size_t)t * ld_src + h * src_hs + src_col0 + 2 * i;
-    T* d = dst + (size_t)t * ld_dst + h * dst_hs + dst_col0 + 2 * i;
-    const float a = to_f<T>(s[0]), b = to_f<T>(s[1]);
+    const int c0 = halves ? i : 2 * i, cb = halves ? i + half : c0 + 1;
+    const T* s = src + (size_t)t * ld_src + h * src_hs + src_col0;
+    T* d = dst + (size_t)t * ld_dst + h * dst_hs + dst_col0;
+    const float a = to_f<T>(s[c0]), b = to_f<T>(s[cb]);
     float sn, cs;
-    sincosf(fp * freq[i], &sn, &cs);
+    rotary_sincos(fp, freq[i], freq_lo ? freq_lo[i] : 0.f, &sn, &cs);
     sn *= mag; cs *= mag;
-    d[0] = from_f<T>(a * cs - b * sn);
-    d[1] = from_f<T>(b * cs + a * sn);
+    d[c0] = from_f<T>(a * cs - b * sn);
+    d[cb] = from_f<T>(b * cs + a * sn);
   }
 }
 
@@ -87,9 +91,9 @@ __global__ void rotary_cols_kernel(T* __restrict__ dst, int ld_dst, int dst_col0
 // out[t, h * o_hs + n] = sum_k A[t, h * a_hs + k] * W[(h * N + n) * K + k]   (* sigmoid(gate[t, h * N + n]))
 constexpr int HG_BM = 64, HG_BN = 64, HG_BK = 16, HG_THREADS = 256, HG_PAD = 4;
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(HG_THREADS)
-head_gemm_kernel(T* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A, int lda, int a_hs,
+head_gemm_kernel(TO* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A, int lda, int a_hs,
                  const T* __restrict__ W, const T* __restrict__ gate, int ldg, int M, int N, int K) {
   __shared__ __align__(16) float As[HG_BK][HG_BM + HG_PAD];
   __shared__ __align__(16) float Bs[HG_BK][HG_BN + HG_PAD];
@@ -138,7 +142,7 @@ head_gemm_kernel(T* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A
       if (n >= N) continue;
       float v = acc[i][j];
       if (gate) v = rnd<T>(v) * (1.f / (1.f + expf(-to_f<T>(gate[(size_t)m * ldg + h * N + n]))));
-      out[(size_t)m * ldo + h * o_hs + n] = from_f<T>(v);
+      out[(size_t)m * ldo + h * o_hs + n] = from_f<TO>(v);
     }
   }
 }
@@ -147,9 +151,9 @@ head_gemm_kernel(T* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A
 // a head and keeps one accumulator per row (up to HV_ROWS rows per launch slice).
 constexpr int HV_ROWS = 8;
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-head_gemv_kernel(T* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A, int lda, int a_hs,
+head_gemv_kernel(TO* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A, int lda, int a_hs,
                  const T* __restrict__ W, const T* __restrict__ gate, int ldg, int M, int N, int K) {
   extern __shared__ float as[];                  // [rows][K] fp32 operand rows of this head
   pdl_launch_dependents();
@@ -192,7 +196,7 @@ head_gemv_kernel(T* __restrict__ out, int ldo, int o_hs, const T* __restrict__ A
       if (lane == 0) {
         const int m = m0 + r;
         if (gate) v = rnd<T>(v) * (1.f / (1.f + expf(-to_f<T>(gate[(size_t)m * ldg + h * N + n]))));
-        out[(size_t)m * ldo + h * o_hs + n] = from_f<T>(v);
+        out[(size_t)m * ldo + h * o_hs + n] = from_f<TO>(v);
       }
     }
   }
@@ -235,7 +239,7 @@ __global__ void concat_cast_kernel(T* __restrict__ out, const float* __restrict_
 
 bool head_gemm_tc_supported(int ldo, int o_gs, int lda, int a_gs, int N, int K, int dtype);
 int head_gemm_tc(void* out, int ldo, int o_gs, const void* A, int lda, int a_gs, const void* W, int n_rows, int heads, int N,
-                 int K, int dtype, int* err_flag, cudaStream_t st);
+                 int K, int out_f32, int dtype, int* err_flag, cudaStream_t st);
 
 }  // namespace pg
 
@@ -246,6 +250,15 @@ extern "C" int pg_latent_prep(void* cq_out, const void* proj, int ld, int dq_col
                               float eps, void* pool, int ld_pool, const int32_t* page_table, int pt_stride,
                               int page_size, const int32_t* tok_slot, const int32_t* tok_pos, int n_tokens, int dtype,
                               void* stream) {
+  return pg_latent_prep_ex(cq_out, proj, ld, dq_col0, q_rank, w_q, dkv_col0, kv_rank, w_kv, rot_dim, freq, nullptr, 0, mag, eps,
+                           pool, ld_pool, page_table, pt_stride, page_size, tok_slot, tok_pos, n_tokens, dtype, stream);
+}
+
+extern "C" int pg_latent_prep_ex(void* cq_out, const void* proj, int ld, int dq_col0, int q_rank, const void* w_q,
+                                 int dkv_col0, int kv_rank, const void* w_kv, int rot_dim, const float* freq,
+                                 const float* freq_lo, int halves, float mag, float eps, void* pool, int ld_pool,
+                                 const int32_t* page_table, int pt_stride, int page_size, const int32_t* tok_slot,
+                                 const int32_t* tok_pos, int n_tokens, int dtype, void* stream) {
   if (n_tokens <= 0) return PG_OK;
   PG_REQUIRE(cq_out && proj && w_q && w_kv && pool && page_table && tok_slot && tok_pos && page_size > 0,
              "latent_prep: operands, pool and token map");
@@ -257,7 +270,8 @@ extern "C" int pg_latent_prep(void* cq_out, const void* proj, int ld, int dq_col
     const int threads = work >= 1024 ? 256 : 128;
     return launch_pdl("latent_prep", latent_prep_kernel<T>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream,
                       (T*)cq_out, (const T*)proj, ld, dq_col0, q_rank, (const T*)w_q, dkv_col0, kv_rank, (const T*)w_kv,
-                      rot_dim, freq, mag, eps, (T*)pool, ld_pool, page_table, pt_stride, page_size, tok_slot, tok_pos);
+                      rot_dim, freq, freq_lo, halves ? 1 : 0, mag, eps, (T*)pool, ld_pool, page_table, pt_stride, page_size,
+                      tok_slot, tok_pos);
   });
   return PG_OK;
 }
@@ -265,6 +279,14 @@ extern "C" int pg_latent_prep(void* cq_out, const void* proj, int ld, int dq_col
 extern "C" int pg_rotary_cols(void* dst, int ld_dst, int dst_col0, int dst_head_stride, const void* src, int ld_src,
                               int src_col0, int src_head_stride, int heads, int rot_dim, const float* freq, float mag,
                               const int32_t* tok_pos, int n_tokens, int dtype, void* stream) {
+  return pg_rotary_cols_ex(dst, ld_dst, dst_col0, dst_head_stride, src, ld_src, src_col0, src_head_stride, heads, rot_dim, freq,
+                           nullptr, 0, mag, tok_pos, n_tokens, dtype, stream);
+}
+
+extern "C" int pg_rotary_cols_ex(void* dst, int ld_dst, int dst_col0, int dst_head_stride, const void* src, int ld_src,
+                                 int src_col0, int src_head_stride, int heads, int rot_dim, const float* freq,
+                                 const float* freq_lo, int halves, float mag, const int32_t* tok_pos, int n_tokens, int dtype,
+                                 void* stream) {
   if (n_tokens <= 0 || rot_dim <= 0) return PG_OK;
   PG_REQUIRE(dst && src && freq && tok_pos && rot_dim % 2 == 0 && heads > 0, "rotary_cols: bad arguments");
   PG_DISPATCH_DTYPE(dtype, T, {
@@ -272,14 +294,14 @@ extern "C" int pg_rotary_cols(void* dst, int ld_dst, int dst_col0, int dst_head_
     const int threads = work >= 512 ? 256 : (work >= 128 ? 128 : 64);
     return launch_pdl("rotary_cols", rotary_cols_kernel<T>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream,
                       (T*)dst, ld_dst, dst_col0, dst_head_stride, (const T*)src, ld_src, src_col0, src_head_stride, heads,
-                      rot_dim, freq, mag, tok_pos);
+                      rot_dim, freq, freq_lo, halves ? 1 : 0, mag, tok_pos);
   });
   return PG_OK;
 }
 
-extern "C" int pg_head_gemm_ex(void* out, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride,
-                               const void* W, const void* gate, int ld_gate, int n_rows, int heads, int N, int K, int impl,
-                               int* err_flag, int dtype, void* stream) {
+static int head_gemm_any(void* out, int out_f32, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride,
+                         const void* W, const void* gate, int ld_gate, int n_rows, int heads, int N, int K, int impl,
+                         int* err_flag, int dtype, void* stream) {
   if (n_rows <= 0) return PG_OK;
   PG_REQUIRE(out && A && W && heads > 0 && N > 0 && K > 0, "head_gemm: bad arguments");
   cudaStream_t st = (cudaStream_t)stream;
@@ -291,7 +313,7 @@ extern "C" int pg_head_gemm_ex(void* out, int ldo, int out_head_stride, const vo
                      ((uintptr_t)gate % 16) == 0 && (long long)n_rows * heads * N < (1ll << 31);
   PG_REQUIRE(impl != 2 || tc_ok, "head_gemm: the tensor-core kernel does not take this problem (N=%d K=%d dtype %d)", N, K, dtype);
   if (impl == 2 || (impl == 0 && tc_ok && n_rows >= tc_min_rows)) {
-    const int rc = head_gemm_tc(out, ldo, out_head_stride, A, lda, a_head_stride, W, n_rows, heads, N, K, dtype, err_flag, st);
+    const int rc = head_gemm_tc(out, ldo, out_head_stride, A, lda, a_head_stride, W, n_rows, heads, N, K, out_f32, dtype, err_flag, st);
     if (rc != PG_OK || !gate) return rc;
     const long long total = (long long)n_rows * heads * (N / 8);
     const int blocks = (int)((total + 255) / 256 < 148 * 32 ? (total + 255) / 256 : 148 * 32);
@@ -301,20 +323,38 @@ extern "C" int pg_head_gemm_ex(void* out, int ldo, int out_head_stride, const vo
     return launch_pdl("head_gate", head_gate_kernel<f16>, dim3(blocks), dim3(256), 0, st, (f16*)out, ldo, out_head_stride,
                       (const f16*)gate, ld_gate, (unsigned)n_rows, (unsigned)heads, (unsigned)N);
   }
-  PG_DISPATCH_DTYPE(dtype, T, {
+  auto run = [&](auto gemv, auto gemm, auto* o, auto* a, auto* w, auto* gt) -> int {
     if (n_rows <= 2 * HV_ROWS && (size_t)HV_ROWS * K * sizeof(float) <= 96 * 1024) {
       const int warps = 8;
       int col_ctas = cdiv(N, warps);
       if (col_ctas * heads > 1184) col_ctas = cdiv(1184, heads);       // about 8 CTAs per SM at most
-      return launch_pdl("head_gemv", head_gemv_kernel<T>, dim3(col_ctas, heads, cdiv(n_rows, HV_ROWS)), dim3(warps * 32),
-                        sizeof(float) * HV_ROWS * (size_t)K, st, (T*)out, ldo, out_head_stride, (const T*)A, lda,
-                        a_head_stride, (const T*)W, (const T*)gate, ld_gate, n_rows, N, K);
+      return launch_pdl("head_gemv", gemv, dim3(col_ctas, heads, cdiv(n_rows, HV_ROWS)), dim3(warps * 32),
+                        sizeof(float) * HV_ROWS * (size_t)K, st, o, ldo, out_head_stride, a, lda, a_head_stride, w, gt, ld_gate,
+                        n_rows, N, K);
     }
-    return launch_pdl("head_gemm", head_gemm_kernel<T>, dim3(cdiv(N, HG_BN), cdiv(n_rows, HG_BM), heads), dim3(HG_THREADS),
-                      0, st, (T*)out, ldo, out_head_stride, (const T*)A, lda, a_head_stride, (const T*)W, (const T*)gate,
-                      ld_gate, n_rows, N, K);
+    return launch_pdl("head_gemm", gemm, dim3(cdiv(N, HG_BN), cdiv(n_rows, HG_BM), heads), dim3(HG_THREADS), 0, st, o, ldo,
+                      out_head_stride, a, lda, a_head_stride, w, gt, ld_gate, n_rows, N, K);
+  };
+  PG_DISPATCH_DTYPE(dtype, T, {
+    if (out_f32)
+      return run(head_gemv_kernel<T, float>, head_gemm_kernel<T, float>, (float*)out, (const T*)A, (const T*)W, (const T*)gate);
+    return run(head_gemv_kernel<T, T>, head_gemm_kernel<T, T>, (T*)out, (const T*)A, (const T*)W, (const T*)gate);
   });
   return PG_OK;
+}
+
+extern "C" int pg_head_gemm_ex(void* out, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride,
+                               const void* W, const void* gate, int ld_gate, int n_rows, int heads, int N, int K, int impl,
+                               int* err_flag, int dtype, void* stream) {
+  return head_gemm_any(out, 0, ldo, out_head_stride, A, lda, a_head_stride, W, gate, ld_gate, n_rows, heads, N, K, impl, err_flag,
+                       dtype, stream);
+}
+
+extern "C" int pg_head_gemm_f32(float* out, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride,
+                                const void* W, int n_rows, int heads, int N, int K, int impl, int* err_flag, int dtype,
+                                void* stream) {
+  return head_gemm_any(out, 1, ldo, out_head_stride, A, lda, a_head_stride, W, nullptr, 0, n_rows, heads, N, K, impl, err_flag,
+                       dtype, stream);
 }
 
 extern "C" int pg_head_gemm(void* out, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride,

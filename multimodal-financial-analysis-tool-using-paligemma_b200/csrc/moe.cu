@@ -3,6 +3,7 @@
 //
 //   pg_moe_route    fp32 router logits, softmax over all routed outputs, top-k on (score + correction), weights =
 //                   score * scale (not renormalised); optional per-token sigmoid gate of a shared expert
+//   pg_moe_route_topk  fp32 router logits with a bias, top-k on the logits, weights = softmax over the chosen ones
 //   pg_moe_sort     pairs whose expert index is < n_experts are grouped by expert (offsets, source rows, position of
 //                   each pair); larger indices are identity experts and take no part in the GEMMs
 //   pg_moe_table_sort  experts picked by token id from a table: the grouping of every such layer of a model in one launch
@@ -185,6 +186,101 @@ __global__ void moe_route_grouped_kernel(int32_t* __restrict__ topk_idx, float* 
   }
   const float inv = 1.f / (wsum + 1e-20f);
   for (int k = lane; k < top; k += 32) topk_w[(size_t)t * top + k] *= inv;
+}
+
+// ------------------------------------------------------------------ router whose weights are a softmax over the chosen logits
+// z = h W_router^T + bias in fp32; the `top` largest z are chosen (ties: lowest index) and weighted by the softmax over the
+// chosen z alone.  A CTA serves TOK tokens: a warp takes an expert and streams its router row once for all of them.
+template <typename T, int TOK>
+__global__ void __launch_bounds__(512)
+moe_route_topk_kernel(int32_t* __restrict__ topk_idx, float* __restrict__ topk_w, const T* __restrict__ h, int ldh,
+                      const T* __restrict__ w_router, const T* __restrict__ bias, int n_tokens, int D, int n_route, int top) {
+  extern __shared__ float smem[];
+  float* hs = smem;                               // [TOK][D]
+  float* z = smem + TOK * D;                      // [TOK][n_route]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int t0 = blockIdx.x * TOK, nt = min(TOK, n_tokens - t0);
+  constexpr int V = Vec<T>::N;
+  const bool vec = D % V == 0 && (reinterpret_cast<uintptr_t>(w_router) & 15) == 0;
+  if (vec && ldh % V == 0 && (reinterpret_cast<uintptr_t>(h) & 15) == 0) {
+    for (int i = threadIdx.x * V; i < TOK * D; i += blockDim.x * V) {
+      const int tt = i / D, k = i - tt * D;
+      float f[V];
+#pragma unroll
+      for (int q = 0; q < V; ++q) f[q] = 0.f;
+      if (tt < nt) unpack<T>(*reinterpret_cast<const uint4*>(h + (size_t)(t0 + tt) * ldh + k), f);
+#pragma unroll
+      for (int q = 0; q < V; ++q) hs[i + q] = f[q];
+    }
+  } else {
+    for (int i = threadIdx.x; i < TOK * D; i += blockDim.x) {
+      const int tt = i / D;
+      hs[i] = tt < nt ? to_f<T>(h[(size_t)(t0 + tt) * ldh + i - tt * D]) : 0.f;
+    }
+  }
+  __syncthreads();
+  for (int e = warp; e < n_route; e += warps) {
+    const T* wr = w_router + (size_t)e * D;
+    float acc[TOK];
+#pragma unroll
+    for (int tt = 0; tt < TOK; ++tt) acc[tt] = 0.f;
+    if (vec) {
+      for (int k = lane * V; k < D; k += 32 * V) {
+        float f[V];
+        unpack<T>(ldg_cached(wr + k), f);
+#pragma unroll
+        for (int tt = 0; tt < TOK; ++tt)
+#pragma unroll
+          for (int q = 0; q < V; q += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(hs + tt * D + k + q);
+            acc[tt] = fmaf(x.x, f[q], acc[tt]); acc[tt] = fmaf(x.y, f[q + 1], acc[tt]);
+            acc[tt] = fmaf(x.z, f[q + 2], acc[tt]); acc[tt] = fmaf(x.w, f[q + 3], acc[tt]);
+          }
+      }
+    } else {
+      for (int k = lane; k < D; k += 32) {
+        const float f = to_f<T>(wr[k]);
+#pragma unroll
+        for (int tt = 0; tt < TOK; ++tt) acc[tt] = fmaf(hs[tt * D + k], f, acc[tt]);
+      }
+    }
+    const float b = bias ? to_f<T>(bias[e]) : 0.f;
+#pragma unroll
+    for (int tt = 0; tt < TOK; ++tt) {
+      const float v = warp_sum(acc[tt]);
+      if (lane == 0) z[tt * n_route + e] = v + b;
+    }
+  }
+  __syncthreads();
+  for (int tt = warp; tt < nt; tt += warps) {      // a warp per token: top-k, then the weights
+    float* zt = z + tt * n_route;
+    const size_t o = (size_t)(t0 + tt) * top;
+    float z0 = 0.f, sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+      unsigned long long best = 0ull;
+      for (int e = lane; e < n_route; e += 32) {
+        const unsigned long long key = argmax_key(zt[e], (unsigned)e);
+        best = key > best ? key : best;
+      }
+#pragma unroll
+      for (int s = 16; s > 0; s >>= 1) {
+        const unsigned long long other = __shfl_xor_sync(0xffffffffu, best, s);
+        best = other > best ? other : best;
+      }
+      const int e = (int)argmax_key_index(best);
+      const float v = argmax_key_value(best);
+      if (k == 0) z0 = v;
+      const float w = expf(v - z0);
+      sum += w;
+      __syncwarp();
+      if (lane == 0) { topk_idx[o + k] = e; topk_w[o + k] = w; zt[e] = -INFINITY; }
+      __syncwarp();
+    }
+    const float inv = 1.f / sum;
+    for (int k = lane; k < top; k += 32) topk_w[o + k] *= inv;
+  }
 }
 
 // ------------------------------------------------------------------ group the pairs by expert (one CTA)
@@ -527,6 +623,24 @@ extern "C" int pg_moe_route_grouped(int32_t* topk_idx, float* topk_w, const void
     return launch_pdl("moe_route_grouped", kern, dim3(n_tokens), dim3(warps * 32), smem, (cudaStream_t)stream, topk_idx,
                       topk_w, (const T*)h, ldh, (const T*)w_router, (const T*)correction, n_tokens, D, n_route, top,
                       n_groups, keep);
+  });
+  return PG_OK;
+}
+
+extern "C" int pg_moe_route_topk(int32_t* topk_idx, float* topk_w, const void* h, int ldh, const void* w_router, const void* bias,
+                                 int n_tokens, int D, int n_route, int top, int dtype, void* stream) {
+  if (n_tokens <= 0) return PG_OK;
+  PG_REQUIRE(topk_idx && topk_w && h && w_router && top >= 1 && top <= n_route && n_route <= 4096,
+             "moe_route_topk: top %d of %d routed outputs", top, n_route);
+  auto smem = [&](int tok) { return sizeof(float) * (size_t)tok * ((size_t)D + n_route); };
+  PG_REQUIRE(smem(1) <= 200 * 1024, "moe_route_topk: D=%d with %d routed outputs does not fit shared memory", D, n_route);
+  PG_DISPATCH_DTYPE(dtype, T, {
+    if (n_tokens >= 296 && smem(8) <= 100 * 1024)
+      return launch_pdl("moe_route_topk", moe_route_topk_kernel<T, 8>, dim3(cdiv(n_tokens, 8)), dim3(256), smem(8), (cudaStream_t)stream,
+                        topk_idx, topk_w, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens, D, n_route, top);
+    return launch_pdl("moe_route_topk", moe_route_topk_kernel<T, 1>, dim3(n_tokens), dim3(n_route >= 16 ? 512 : 256), smem(1),
+                      (cudaStream_t)stream, topk_idx, topk_w, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens, D,
+                      n_route, top);
   });
   return PG_OK;
 }

@@ -30,6 +30,7 @@ struct MoeParams {
   // reads its operand at columns e * a_gs of the token rows (the A map covers the token-major matrix) and writes
   // columns e * o_gs of them.
   int group_rows, a_gs, o_gs;
+  int out_f32;     // one product per output: the accumulators are stored as fp32, unrounded (ldo and o_gs count floats)
 };
 
 // Every wait of this kernel is bounded: if the roles ever disagreed about the tile sequence (the offsets are data),
@@ -198,6 +199,12 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
 #pragma unroll
           for (int j0 = 0; j0 < 32; j0 += 8) {
             if (n0 + j0 >= p.N) break;  // N is a multiple of 8 (checked on the host)
+            if (!DUAL && p.out_f32) {
+              float4* d = reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + o_at + n0 + j0);
+              d[0] = make_float4(v[j0], v[j0 + 1], v[j0 + 2], v[j0 + 3]);
+              d[1] = make_float4(v[j0 + 4], v[j0 + 5], v[j0 + 6], v[j0 + 7]);
+              continue;
+            }
             float o[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
@@ -277,7 +284,7 @@ int moe_gemm_tc(void* out, int ldo, const void* A, int lda, const int32_t* row_m
   PG_REQUIRE(tc::make_map_2d(&ma, A, n_pairs, K, lda, tc::MG_BM, bf) &&
                  tc::make_map_2d(&mw, W, (long long)n_experts * rows_per_expert, K, K, bn, bf),
              "moe_gemm_tc: cuTensorMapEncodeTiled failed (rows=%d N=%d K=%d)", n_pairs, N, K);
-  tc::MoeParams p = {out, offsets, n_experts, N, K, ldo, err_flag, act, limit, 0, 0, 0};
+  tc::MoeParams p = {out, offsets, n_experts, N, K, ldo, err_flag, act, limit, 0, 0, 0, 0};
   const int max_tiles = (cdiv(n_pairs, tc::MG_BM) + n_experts) * cdiv(N, bn);
 #define PG_MOE(D, B) return bf ? tc::launch_moe<bf16, D, B>(ma, mw, p, max_tiles, st) : tc::launch_moe<f16, D, B>(ma, mw, p, max_tiles, st)
   if (swiglu) { if (bn == 128) { PG_MOE(true, 128); } PG_MOE(true, 64); }
@@ -296,7 +303,7 @@ bool head_gemm_tc_supported(int ldo, int o_gs, int lda, int a_gs, int N, int K, 
 }
 
 int head_gemm_tc(void* out, int ldo, int o_gs, const void* A, int lda, int a_gs, const void* W, int n_rows, int heads, int N,
-                 int K, int dtype, int* err_flag, cudaStream_t st) {
+                 int K, int out_f32, int dtype, int* err_flag, cudaStream_t st) {
   PG_REQUIRE(((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0 && ((uintptr_t)out % 16) == 0,
              "head_gemm_tc: operands must be 16-byte aligned");
   const bool bf = dtype == PG_BF16;
@@ -305,7 +312,7 @@ int head_gemm_tc(void* out, int ldo, int o_gs, const void* A, int lda, int a_gs,
   PG_REQUIRE(tc::make_map_2d(&ma, A, n_rows, lda, lda, tc::MG_BM, bf) &&
                  tc::make_map_2d(&mw, W, (long long)heads * N, K, K, bn, bf),
              "head_gemm_tc: cuTensorMapEncodeTiled failed (rows=%d N=%d K=%d)", n_rows, N, K);
-  tc::MoeParams p = {out, nullptr, heads, N, K, ldo, err_flag, PG_GLU_NONE, 0.f, n_rows, a_gs, o_gs};
+  tc::MoeParams p = {out, nullptr, heads, N, K, ldo, err_flag, PG_GLU_NONE, 0.f, n_rows, a_gs, o_gs, out_f32};
   const int max_tiles = heads * cdiv(n_rows, tc::MG_BM) * cdiv(N, bn);
   if (bn == 128) return bf ? tc::launch_moe<bf16, false, 128>(ma, mw, p, max_tiles, st) : tc::launch_moe<f16, false, 128>(ma, mw, p, max_tiles, st);
   return bf ? tc::launch_moe<bf16, false, 64>(ma, mw, p, max_tiles, st) : tc::launch_moe<f16, false, 64>(ma, mw, p, max_tiles, st);

@@ -1,5 +1,6 @@
 // Recurrent mixers for ragged token batches: the generalised delta rule with a per-channel decay, and lightning
-// attention (linear attention with a constant decay per head; described at its kernel below).
+// attention (linear attention with a constant decay per head; described at its kernel below) with its relatives: retention,
+// the state-space scan (a decay per token) and gated linear attention (a decay per token and key channel).
 //
 // Per head, with a state S [dim x dim] (key channel i, value column j) kept in fp32 per sequence slot:
 //     u   = k / sqrt(sum(k^2) + key_eps)
@@ -301,11 +302,76 @@ __global__ void lightning_prep_kernel(float* __restrict__ rec, const T* __restri
   }
 }
 
+// Gated linear attention runs on the same recurrence with a decay per key channel: a = sigmoid(z)^(1/tau), z = W2 inner + b2
+// with `inner` the decay's low-rank projection.  The W2 product, the logarithm and the exponential are fp32.  A CTA takes
+// PREP_TOK tokens; a thread owns a key channel and walks its W2 row once for all of them.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gla_prep_kernel(float* __restrict__ rec, const T* __restrict__ proj, int ld, int q_col0, int k_col0, int v_col0, int a_col0,
+                int rank, const T* __restrict__ w2, const T* __restrict__ b2, float q_scale, float inv_tau, int n_tokens,
+                int heads, int dim, int vdim, int dp, int vp) {
+  extern __shared__ float lo[];                     // [PREP_TOK][rank]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * PREP_TOK, nt = min(PREP_TOK, n_tokens - t0), rs = 3 * dp + vp;
+  for (int idx = threadIdx.x; idx < PREP_TOK * rank; idx += blockDim.x) {
+    const int tt = idx / rank, j = idx - tt * rank;
+    lo[idx] = tt < nt ? to_f<T>(proj[(size_t)(t0 + tt) * ld + a_col0 + j]) : 0.f;
+  }
+  __syncthreads();
+  constexpr int V = Vec<T>::N;
+  const bool vec = (rank % V) == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0;
+  // blockIdx.y cuts the columns into slices (a handful of tokens: more CTAs than token groups)
+  const int n_key = heads * dp, k_per = (n_key + gridDim.y - 1) / gridDim.y, k_end = min(n_key, (int)(blockIdx.y + 1) * k_per);
+  for (int c = blockIdx.y * k_per + threadIdx.x; c < k_end; c += blockDim.x) {
+    const int h = c / dp, i = c - h * dp, ch = h * dim + i;
+    float z[PREP_TOK];
+    const bool in = i < dim;                        // the padding channels of a record are zero
+    const float z0 = in ? to_f<T>(b2[ch]) : 0.f;
+#pragma unroll
+    for (int tt = 0; tt < PREP_TOK; ++tt) z[tt] = z0;
+    if (in) {
+      const T* wr = w2 + (size_t)ch * rank;
+      if (vec) {
+        for (int j = 0; j < rank; j += V) {
+          float f[V];
+          unpack<T>(*reinterpret_cast<const uint4*>(wr + j), f);
+#pragma unroll
+          for (int tt = 0; tt < PREP_TOK; ++tt)
+#pragma unroll
+            for (int k = 0; k < V; ++k) z[tt] = fmaf(f[k], lo[tt * rank + j + k], z[tt]);
+        }
+      } else {
+        for (int j = 0; j < rank; ++j) {
+          const float f = to_f<T>(wr[j]);
+#pragma unroll
+          for (int tt = 0; tt < PREP_TOK; ++tt) z[tt] = fmaf(f, lo[tt * rank + j], z[tt]);
+        }
+      }
+    }
+#pragma unroll
+    for (int tt = 0; tt < PREP_TOK; ++tt) {
+      if (tt >= nt) break;
+      const T* row = proj + (size_t)(t0 + tt) * ld;
+      float* o = rec + ((size_t)(t0 + tt) * heads + h) * rs + i;
+      o[0] = in ? to_f<T>(row[q_col0 + ch]) * q_scale : 0.f;
+      o[dp] = in ? to_f<T>(row[k_col0 + ch]) : 0.f;
+      o[2 * dp] = in ? expf((fminf(z[tt], 0.f) - log1pf(expf(-fabsf(z[tt])))) * inv_tau) : 0.f;
+    }
+  }
+  const int n_val = heads * vp, v_per = (n_val + gridDim.y - 1) / gridDim.y, v_end = min(n_val, (int)(blockIdx.y + 1) * v_per);
+  for (int c = blockIdx.y * v_per + threadIdx.x; c < v_end; c += blockDim.x) {
+    const int h = c / vp, i = c - h * vp;
+    for (int tt = 0; tt < nt; ++tt)
+      rec[((size_t)(t0 + tt) * heads + h) * rs + 3 * dp + i] =
+          i < vdim ? to_f<T>(proj[(size_t)(t0 + tt) * ld + v_col0 + h * vdim + i]) : 0.f;
+  }
+}
+
 // Retention (linear attention with rotary positions in place of activations) runs on the same recurrence: its records
 // are written by retention_prep_kernel below.  The first rot_dims columns of every q and k head are turned in pairs
 // (i, i + rot_dims / 2), or (2i, 2i + 1) when interleaved, by position * freq[i]; k is multiplied by k_scale after the
-// rotation; v passes.  freq holds (high, low) float pairs: the angle's rounding error and the low part enter as a first-
-// order correction, so that far positions keep full fp32 accuracy.  One CTA per token: the token's sines and cosines
+// rotation; v passes.  freq holds (high, low) float pairs (rotary_sincos).  One CTA per token: the token's sines and cosines
 // once into shared memory (the heads share them), then records four columns at a time.
 template <typename T>
 __global__ void retention_prep_kernel(float* __restrict__ rec, const T* __restrict__ proj, int ld, int q_col0, int k_col0,
@@ -319,10 +385,9 @@ __global__ void retention_prep_kernel(float* __restrict__ rec, const T* __restri
   const float p = (float)tok_pos[t];
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const float2 f = freq[i];
-    const float a = p * f.x, d = fmaf(p, f.x, -a) + p * f.y;   // the exact angle is a + d
     float s, c;
-    sincosf(a, &s, &c);
-    cs[i] = make_float2(c - s * d, s + c * d);
+    rotary_sincos(p, f.x, f.y, &s, &c);
+    cs[i] = make_float2(c, s);
   }
   __syncthreads();
   const T* row = proj + t * ld;
@@ -391,27 +456,31 @@ __global__ void retention_prep_kernel(float* __restrict__ rec, const T* __restri
   }
 }
 
-//                                       TD (decay per token): the record carries four more floats [decay, 0, 0, 0] after
-//                                       the values and the decay of a token comes from there instead of decay[h];
+//                                       DK (where the decay comes from): DECAY_HEAD decay[h]; DECAY_TOKEN: the record carries
+//                                       four more floats [decay, 0, 0, 0] after the values; DECAY_CHANNEL: a vector of dp
+//                                       decays between key and values, one per key channel (gated linear attention);
 //                                       skip (may be NULL): skip[h] * v is added to the output (the state-space
 //                                       mixer's direct term, with v its unscaled input).
-template <int DMAX, int RG, int CH, bool TD>
+enum { DECAY_HEAD = 0, DECAY_TOKEN = 1, DECAY_CHANNEL = 2 };
+
+template <int DMAX, int RG, int CH, int DK>
 __global__ void __launch_bounds__(256)
 lightning_kernel(float* __restrict__ out, float* __restrict__ state, const float* __restrict__ rec,
                  const float* __restrict__ decay, const float* __restrict__ skip, const int32_t* __restrict__ segs,
                  int heads, int dim, int vdim, int dp, int vp) {
   constexpr int NG = DMAX / (4 * RG);               // groups of four rows per thread (RG lanes share a value column)
-  extern __shared__ __align__(16) float sh[];       // [2][CH][q DMAX | k DMAX | v VT]
+  extern __shared__ __align__(16) float sh[];       // [2][CH][q DMAX | k DMAX | (decays DMAX) | v VT | (decay)]
   pdl_launch_dependents();
   pdl_wait();
   const int32_t* sg = segs + 3 * (size_t)blockIdx.x;
   const int slot = sg[0], row0 = sg[1], n = sg[2];
   if (n <= 0) return;
-  constexpr int XP = TD ? 4 : 0;
-  const int VT = blockDim.x / RG, RSZ = 2 * DMAX + VT + XP, rs = 2 * dp + vp + XP;
+  constexpr bool TD = DK == DECAY_TOKEN, CD = DK == DECAY_CHANNEL;
+  constexpr int XP = TD ? 4 : 0, NV = CD ? 3 : 2;   // NV: vectors of key width in a record
+  const int VT = blockDim.x / RG, RSZ = NV * DMAX + VT + XP, rs = NV * dp + vp + XP;
   const int h = blockIdx.y, j0 = blockIdx.z * VT, jl = threadIdx.x / RG, j = j0 + jl, rg = threadIdx.x % RG;
   const bool live = j < vdim;
-  const float lam_h = TD ? 0.f : decay[h], skip_h = skip ? skip[h] : 0.f;
+  const float lam_h = DK == DECAY_HEAD ? decay[h] : 0.f, skip_h = skip ? skip[h] : 0.f;
   for (int idx = threadIdx.x; idx < 2 * CH * RSZ; idx += blockDim.x) sh[idx] = 0.f;   // padding the copies never write
   float S[NG * 4];
   float* st = state + ((size_t)slot * heads + h) * dim * vdim;
@@ -423,7 +492,7 @@ lightning_kernel(float* __restrict__ out, float* __restrict__ state, const float
       S[m * 4 + e] = (live && i < dim) ? st[(size_t)i * vdim + j] : 0.f;
     }
   __syncthreads();
-  const int qk_pieces = dp / 4, v_pieces = min(VT, vp - j0) / 4, pieces = 2 * qk_pieces + v_pieces + (TD ? 1 : 0);
+  const int qk_pieces = dp / 4, v_pieces = min(VT, vp - j0) / 4, pieces = NV * qk_pieces + v_pieces + (TD ? 1 : 0);
   auto fetch = [&](int t0, int buf) {               // records of tokens [t0, t0 + CH) of this head -> buffer buf
     const int nt = min(CH, n - t0);
     for (int idx = threadIdx.x; idx < nt * pieces; idx += blockDim.x) {
@@ -432,8 +501,9 @@ lightning_kernel(float* __restrict__ out, float* __restrict__ state, const float
       float* dst = sh + ((size_t)buf * CH + tt) * RSZ;
       if (pc < qk_pieces) cp_async16(dst + pc * 4, src + pc * 4);
       else if (pc < 2 * qk_pieces) cp_async16(dst + DMAX + (pc - qk_pieces) * 4, src + dp + (pc - qk_pieces) * 4);
-      else if (pc < 2 * qk_pieces + v_pieces) cp_async16(dst + 2 * DMAX + (pc - 2 * qk_pieces) * 4, src + 2 * dp + j0 + (pc - 2 * qk_pieces) * 4);
-      else cp_async16(dst + 2 * DMAX + VT, src + 2 * dp + vp);
+      else if (CD && pc < 3 * qk_pieces) cp_async16(dst + 2 * DMAX + (pc - 2 * qk_pieces) * 4, src + 2 * dp + (pc - 2 * qk_pieces) * 4);
+      else if (pc < NV * qk_pieces + v_pieces) cp_async16(dst + NV * DMAX + (pc - NV * qk_pieces) * 4, src + NV * dp + j0 + (pc - NV * qk_pieces) * 4);
+      else cp_async16(dst + NV * DMAX + VT, src + NV * dp + vp);
     }
     cp_async_commit();
   };
@@ -446,19 +516,22 @@ lightning_kernel(float* __restrict__ out, float* __restrict__ state, const float
 #pragma unroll 2
     for (int tt = 0; tt < nt; ++tt) {
       const float* r = sh + ((size_t)buf * CH + tt) * RSZ;
-      const float vj = r[2 * DMAX + jl];
-      const float lam = TD ? r[2 * DMAX + VT] : lam_h;
+      const float vj = r[NV * DMAX + jl];
+      const float lam = TD ? r[NV * DMAX + VT] : lam_h;
       const float* qr = r + 4 * rg;
       const float* kr = r + DMAX + 4 * rg;
+      const float* ar = r + 2 * DMAX + 4 * rg;       // decays per key channel (CD)
       float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
 #pragma unroll
       for (int m = 0; m < NG; ++m) {
         const float4 k4 = *reinterpret_cast<const float4*>(kr + 4 * RG * m);
         const float4 q4 = *reinterpret_cast<const float4*>(qr + 4 * RG * m);
-        S[4 * m] = fmaf(k4.x, vj, lam * S[4 * m]);
-        S[4 * m + 1] = fmaf(k4.y, vj, lam * S[4 * m + 1]);
-        S[4 * m + 2] = fmaf(k4.z, vj, lam * S[4 * m + 2]);
-        S[4 * m + 3] = fmaf(k4.w, vj, lam * S[4 * m + 3]);
+        float4 a4 = make_float4(lam, lam, lam, lam);
+        if (CD) a4 = *reinterpret_cast<const float4*>(ar + 4 * RG * m);
+        S[4 * m] = fmaf(k4.x, vj, a4.x * S[4 * m]);
+        S[4 * m + 1] = fmaf(k4.y, vj, a4.y * S[4 * m + 1]);
+        S[4 * m + 2] = fmaf(k4.z, vj, a4.z * S[4 * m + 2]);
+        S[4 * m + 3] = fmaf(k4.w, vj, a4.w * S[4 * m + 3]);
         o0 = fmaf(q4.x, S[4 * m], o0); o1 = fmaf(q4.y, S[4 * m + 1], o1);
         o2 = fmaf(q4.z, S[4 * m + 2], o2); o3 = fmaf(q4.w, S[4 * m + 3], o3);
       }
@@ -481,7 +554,7 @@ lightning_kernel(float* __restrict__ out, float* __restrict__ state, const float
 }
 
 template <int DMAX, int RG, int CH>
-static int launch_lightning(float* out, float* state, const float* rec, const float* decay, const float* skip, bool td,
+static int launch_lightning(float* out, float* state, const float* rec, const float* decay, const float* skip, int dk,
                             const int32_t* segs, int n_segs, int heads, int dim, int vdim, cudaStream_t st) {
   const int dp = (dim + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4;
   // value columns per CTA: as many as 256 threads hold for prompt-sized work (few fat CTAs, about one per SM, beat
@@ -490,16 +563,18 @@ static int launch_lightning(float* out, float* state, const float* rec, const fl
   while (vt > 8 && (vt / 2 >= vdim || (long long)n_segs * heads * cdiv(vdim, vt) < 100)) vt /= 2;
   static const int vt_env = env_int("PG_LIGHTNING_VT", 0);
   if (vt_env >= 8 && vt_env <= 256 / RG && (vt_env & (vt_env - 1)) == 0) vt = vt_env;
-  const size_t smem = sizeof(float) * 2 * CH * (2 * DMAX + vt + (td ? 4 : 0));
+  const size_t smem = sizeof(float) * 2 * CH * ((dk == DECAY_CHANNEL ? 3 : 2) * DMAX + vt + (dk == DECAY_TOKEN ? 4 : 0));
   // An ordinary launch, not a programmatic dependent one: CTAs that become resident while the preceding kernel still
   // fills the machine are placed on the few SMs with room, and a recurrence of a few hundred long-lived CTAs then runs
   // on a fraction of the GPU (measured at 4 x 2048 tokens, 8 heads of 128: 2.06 ms against 0.88 ms).
-  if (td)
-    lightning_kernel<DMAX, RG, CH, true><<<dim3(n_segs, heads, cdiv(vdim, vt)), dim3(vt * RG), smem, st>>>(
-        out, state, rec, decay, skip, segs, heads, dim, vdim, dp, vp);
-  else
-    lightning_kernel<DMAX, RG, CH, false><<<dim3(n_segs, heads, cdiv(vdim, vt)), dim3(vt * RG), smem, st>>>(
-        out, state, rec, decay, skip, segs, heads, dim, vdim, dp, vp);
+  auto kern = dk == DECAY_CHANNEL ? lightning_kernel<DMAX, RG, CH, DECAY_CHANNEL>
+                                  : (dk == DECAY_TOKEN ? lightning_kernel<DMAX, RG, CH, DECAY_TOKEN> : lightning_kernel<DMAX, RG, CH, DECAY_HEAD>);
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    set_error("lightning: cannot reserve %zu B of shared memory", smem);
+    cudaGetLastError();
+    return PG_ERR_CUDA;
+  }
+  kern<<<dim3(n_segs, heads, cdiv(vdim, vt)), dim3(vt * RG), smem, st>>>(out, state, rec, decay, skip, segs, heads, dim, vdim, dp, vp);
   return check_launch("lightning");
 }
 
@@ -613,10 +688,9 @@ extern "C" int pg_lightning_attention(float* out, float* state, const float* rec
   return pg_lightning_attention_ex(out, state, rec, decay, nullptr, segs, n_segs, heads, dim, vdim, stream);
 }
 
-extern "C" int pg_lightning_attention_ex(float* out, float* state, const float* rec, const float* decay, const float* skip,
-                                         const int32_t* segs, int n_segs, int heads, int dim, int vdim, void* stream) {
+static int lightning_any(float* out, float* state, const float* rec, const float* decay, const float* skip, int td,
+                         const int32_t* segs, int n_segs, int heads, int dim, int vdim, void* stream) {
   if (n_segs <= 0) return PG_OK;
-  const bool td = decay == nullptr;                 // no constant decay: the records carry one per token
   PG_REQUIRE(out && state && rec && segs, "lightning_attention: bad arguments");
   PG_REQUIRE(dim > 0 && dim <= 256 && vdim > 0, "lightning_attention: key size %d (1..256), value size %d", dim, vdim);
   cudaStream_t st = (cudaStream_t)stream;
@@ -633,4 +707,37 @@ extern "C" int pg_lightning_attention_ex(float* out, float* state, const float* 
     return deep ? launch_lightning<128, 8, 16>(out, state, rec, decay, skip, td, segs, n_segs, heads, dim, vdim, st)
                 : launch_lightning<128, 8, 8>(out, state, rec, decay, skip, td, segs, n_segs, heads, dim, vdim, st);
   return launch_lightning<256, 16, 4>(out, state, rec, decay, skip, td, segs, n_segs, heads, dim, vdim, st);
+}
+
+extern "C" int pg_lightning_attention_ex(float* out, float* state, const float* rec, const float* decay, const float* skip,
+                                         const int32_t* segs, int n_segs, int heads, int dim, int vdim, void* stream) {
+  // no constant decay: the records carry one per token
+  return lightning_any(out, state, rec, decay, skip, decay ? DECAY_HEAD : DECAY_TOKEN, segs, n_segs, heads, dim, vdim, stream);
+}
+
+extern "C" int pg_gla_attention(float* out, float* state, const float* rec, const int32_t* segs, int n_segs, int heads, int dim,
+                                int vdim, void* stream) {
+  return lightning_any(out, state, rec, nullptr, nullptr, DECAY_CHANNEL, segs, n_segs, heads, dim, vdim, stream);
+}
+
+extern "C" long long pg_gla_record_floats(int n_tokens, int heads, int dim, int vdim) {
+  return (long long)n_tokens * heads * (3 * ((dim + 3) / 4 * 4) + (vdim + 3) / 4 * 4);
+}
+
+extern "C" int pg_gla_prep(float* rec, const void* proj, int ld, int q_col0, int k_col0, int v_col0, int a_col0, int rank,
+                           const void* w2, const void* b2, float q_scale, float inv_tau, int n_tokens, int heads, int dim,
+                           int vdim, int dtype, void* stream) {
+  if (n_tokens <= 0) return PG_OK;
+  PG_REQUIRE(rec && proj && w2 && b2 && rank > 0 && heads > 0 && dim > 0 && vdim > 0, "gla_prep: bad arguments");
+  const int dp = (dim + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4;
+  const size_t smem = sizeof(float) * PREP_TOK * (size_t)rank;
+  PG_REQUIRE(smem <= 200 * 1024, "gla_prep: an inner projection of %d columns does not fit shared memory", rank);
+  PG_DISPATCH_DTYPE(dtype, T, {
+    const int work = heads * (dp > vp ? dp : vp), threads = work >= 256 ? 256 : 128;
+    const int slices = n_tokens <= 64 ? cdiv(heads * dp, threads) : 1;
+    return launch_pdl("gla_prep", gla_prep_kernel<T>, dim3(cdiv(n_tokens, PREP_TOK), slices), dim3(threads), smem,
+                      (cudaStream_t)stream, rec, (const T*)proj, ld, q_col0, k_col0, v_col0, a_col0, rank, (const T*)w2,
+                      (const T*)b2, q_scale, inv_tau, n_tokens, heads, dim, vdim, dp, vp);
+  });
+  return PG_OK;
 }

@@ -137,9 +137,26 @@ SIGNATURES = {
     "pg_attention_ragged_tc_ok8": [_i, _i, _i, _i, _i, _i, _i],
     "pg_attention_ragged_tc_capped": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _ll, _vp, _i, _i, _vp, _i, _i, _i, _i,
                                       _i, _i, _f, _i, _i, _i, _vp, _i, _vp, _vp, _f, _f, _i, _vp, _i, _f, _vp, _i, _vp],
+    # hyper-connections, gated linear attention, convolved queries and keys, gated linear recurrent unit
+    "pg_hyper_connect": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _vp, _vp, _f, _f, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp,
+                         _vp, _i, _i, _vp, _i, _vp],
+    "pg_gla_record_floats": [_i, _i, _i, _i],
+    "pg_gla_prep": [_vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _f, _i, _i, _i, _i, _i, _vp],
+    "pg_gla_attention": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "pg_conv_qk_append": [_vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _f, _vp, _i, _vp, _vp, _vp, _i, _i, _vp,
+                          _vp, _i, _i, _vp],
+    "pg_lru_conv": [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _vp],
+    "pg_lru_ws_floats": [_i, _i, _i],
+    "pg_lru_scan": [_vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _i, _i, _i, _i, _vp, _i, _i, _vp],
+    "pg_moe_route_topk": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "pg_head_gemm_f32": [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
+    "pg_latent_prep_ex": [_vp, _vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _i, _f, _f, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i,
+                          _vp],
+    "pg_rotary_cols_ex": [_vp, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _vp, _i, _i, _vp],
 }
 _RESTYPE = {"pg_last_error": C.c_char_p, "pg_launch_count": _ull, "pg_decode_attention_ws_floats": _ll,
-            "pg_delta_record_floats": _ll, "pg_lightning_record_floats": _ll, "pg_ssm_record_floats": _ll}
+            "pg_delta_record_floats": _ll, "pg_lightning_record_floats": _ll, "pg_ssm_record_floats": _ll,
+            "pg_gla_record_floats": _ll, "pg_lru_ws_floats": _ll}
 
 _lib = None
 

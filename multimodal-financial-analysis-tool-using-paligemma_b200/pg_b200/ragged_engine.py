@@ -76,6 +76,12 @@ class RotaryCfg:
         return f, mag
 
 
+def rotary_pairs(rot: RotaryCfg) -> torch.Tensor:
+    """The frequencies as (high, low) fp32 pairs [dims / 2, 2]: high + low is the float64 value to 48 bits."""
+    f, _ = rot.table()
+    hi = f.to(torch.float32)
+    return torch.stack([hi, (f - hi.to(torch.float64)).to(torch.float32)], 1).contiguous()
+
 
 @dataclass
 class LoopCfg:

@@ -48,7 +48,8 @@ import torch
 
 from . import _cabi as cabi
 from ._cabi import ptr
-from .ragged_engine import LoopCfg, RaggedEngine, RotaryCfg, Run, StepInputs, _stack_rows, layer_runs, loop_cfg
+from .ragged_engine import (LoopCfg, RaggedEngine, RotaryCfg, Run, StepInputs, _stack_rows, layer_runs, loop_cfg,
+                            rotary_pairs)
 from .registry import register
 
 
@@ -154,13 +155,6 @@ class RanesunConfig:
         return RanesunConfig(vocab=int(cfg["vocab"]), width=int(cfg["width"]), eps=float((cfg.get("norm") or {})["eps"]),
                              logit_scale=float(cfg.get("logit_scale", 1.0)), layers=layers,
                              loop=loop_cfg(cfg.get("loop"), len(layers)))
-
-
-def rotary_pairs(rot: RotaryCfg) -> torch.Tensor:
-    """The frequencies as (high, low) fp32 pairs [dims / 2, 2]: high + low is the float64 value to 48 bits."""
-    f, _ = rot.table()
-    hi = f.to(torch.float32)
-    return torch.stack([hi, (f - hi.to(torch.float64)).to(torch.float32)], 1).contiguous()
 
 
 @register("Ranesun")

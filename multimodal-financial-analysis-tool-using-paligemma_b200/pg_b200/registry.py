@@ -36,6 +36,7 @@ def _load_builtin() -> None:
     from . import birizen  # noqa: F401  (registers itself)
     from . import gogivik  # noqa: F401
     from . import mubasun  # noqa: F401
+    from . import mutirax  # noqa: F401
     from . import ninisun  # noqa: F401
     from . import ranesun  # noqa: F401
     from . import engine   # noqa: F401
