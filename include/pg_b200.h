@@ -639,20 +639,20 @@ int pg_attention_ragged_tc_capped(void* out, int ld_out, const void* q, int ld_q
  *   (W2 [heads * dim][rank], b2 [heads * dim]; fp32).  rec holds pg_gla_record_floats() floats; state, segs, out as for
  *   pg_lightning_attention.
  * pg_conv_qk_append: per token, from the fused projection row: q and k pass a causal convolution over time per channel
- *   (conv: device fp32 [taps][columns from q_col0 to the end of k], last row = the current token), v = k right after it;
+ *   (conv: model dtype [taps][columns from q_col0 to the end of k], last row = the current token), v = k right after it;
  *   q and k are divided by their root mean square over all heads' columns and multiplied by q_w / k_w (NULL: no norm), then
  *   rotated (pairs (i, i + rot_dims / 2) of every head, freq: device (high, low) float pairs).  q to q_out (packed), k and v to
  *   the paged pools (rows of n_kv_heads * dim).  state: [slots][state_len][state_cols] fp32, column 0 = projection column
  *   q_col0, as pg_time_conv_state keeps it (state_len >= taps - 1; entry state_len - 1 the most recent).
  * pg_lru_conv: u = conv(x + x_bias) + conv_b per channel (model dtype, packed), zeros before position 0; the state holds
- *   projected values without the bias.  conv: device fp32 [taps][width].
+ *   projected values without the bias.  conv: model dtype [taps][width].
  * pg_lru_scan: r = sigmoid(z_r + r_bias), i = sigmoid(z_i + i_bias), log a = -c r softplus(lam),
  *   S <- a S + sqrt(1 - a^2) i u, out = S * gelu_tanh(y + y_bias), all fp32 with one rounding.  z: device fp32
  *   [n_tokens][blocks][r: width / blocks | i: width / blocks]; state [slots][width] fp32; segs as for pg_delta_rule, the
- *   non-empty ones in row order before the empty ones.  ws: pg_lru_ws_floats() floats for the chunked form.  impl 0 picks, 1 =
- *   token by token, 2 = chunked.
+ *   non-empty ones in row order before the empty ones.  ws: pg_lru_ws_floats() floats for the chunked form, which overwrites z.
+ *   impl 0 picks, 1 = token by token, 2 = chunked.
  * pg_moe_route_topk: z = h W_router^T + bias in fp32 (bias may be NULL), the `top` largest z are chosen (ties: lowest index),
- *   topk_w = softmax over the chosen z.
+ *   topk_w = softmax over the chosen z.  logits (device fp32 [n_tokens][n_route], may be NULL): h W_router^T, computed already.
  * pg_head_gemm_f32: pg_head_gemm_ex without a gate and with fp32 output (ldo, out_head_stride in floats).
  * pg_latent_prep_ex / pg_rotary_cols_ex: with the low parts of the frequencies (freq_lo, may be NULL) and, halves != 0, pairs
  *   (i, i + rot_dim / 2). */
@@ -667,19 +667,19 @@ int pg_gla_prep(float* rec, const void* proj, int ld, int q_col0, int k_col0, in
 int pg_gla_attention(float* out, float* state, const float* rec, const int32_t* segs, int n_segs, int heads, int dim, int vdim,
                      void* stream);
 int pg_conv_qk_append(void* q_out, const void* proj, int ld, int q_col0, int n_heads, int k_col0, int n_kv_heads, int dim,
-                      const float* conv, int taps, const float* state, int state_len, int state_cols, const void* q_w,
+                      const void* conv, int taps, const float* state, int state_len, int state_cols, const void* q_w,
                       const void* k_w, float eps, const float* freq, int rot_dims, void* k_pool, void* v_pool,
                       const int32_t* page_table, int pt_stride, int page_size, const int32_t* tok_slot, const int32_t* tok_pos,
                       int n_tokens, int dtype, void* stream);
-int pg_lru_conv(void* u, const void* proj, int ld, int x_col0, const void* x_bias, const float* conv, const void* conv_b, int taps,
+int pg_lru_conv(void* u, const void* proj, int ld, int x_col0, const void* x_bias, const void* conv, const void* conv_b, int taps,
                 const float* state, int state_len, int state_cols, const int32_t* tok_slot, const int32_t* tok_pos, int n_tokens,
                 int width, int dtype, void* stream);
 long long pg_lru_ws_floats(int n_tokens, int n_segs, int width);
-int pg_lru_scan(void* out, int ld_out, float* state, const float* z, const void* u, const void* y, int ld_y, const void* y_bias,
+int pg_lru_scan(void* out, int ld_out, float* state, float* z, const void* u, const void* y, int ld_y, const void* y_bias,
                 const void* r_bias, const void* i_bias, const float* lam, float c, const int32_t* segs, int n_segs, int n_tokens,
                 int width, int blocks, float* ws, int impl, int dtype, void* stream);
-int pg_moe_route_topk(int32_t* topk_idx, float* topk_w, const void* h, int ldh, const void* w_router, const void* bias, int n_tokens,
-                      int D, int n_route, int top, int dtype, void* stream);
+int pg_moe_route_topk(int32_t* topk_idx, float* topk_w, const float* logits, const void* h, int ldh, const void* w_router,
+                      const void* bias, int n_tokens, int D, int n_route, int top, int dtype, void* stream);
 int pg_head_gemm_f32(float* out, int ldo, int out_head_stride, const void* A, int lda, int a_head_stride, const void* W, int n_rows,
                      int heads, int N, int K, int impl, int* err_flag, int dtype, void* stream);
 int pg_latent_prep_ex(void* cq_out, const void* proj, int ld, int dq_col0, int q_rank, const void* w_q, int dkv_col0, int kv_rank,

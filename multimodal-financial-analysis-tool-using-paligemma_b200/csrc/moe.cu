@@ -191,20 +191,25 @@ __global__ void moe_route_grouped_kernel(int32_t* __restrict__ topk_idx, float* 
 // ------------------------------------------------------------------ router whose weights are a softmax over the chosen logits
 // z = h W_router^T + bias in fp32; the `top` largest z are chosen (ties: lowest index) and weighted by the softmax over the
 // chosen z alone.  A CTA serves TOK tokens: a warp takes an expert and streams its router row once for all of them.
+// With `logits` (fp32 [n_tokens][n_route], before the bias: a GEMM of the step left them) only the choice is made here.
 template <typename T, int TOK>
 __global__ void __launch_bounds__(512)
-moe_route_topk_kernel(int32_t* __restrict__ topk_idx, float* __restrict__ topk_w, const T* __restrict__ h, int ldh,
+moe_route_topk_kernel(int32_t* __restrict__ topk_idx, float* __restrict__ topk_w, const float* __restrict__ logits,
+                      const T* __restrict__ h, int ldh,
                       const T* __restrict__ w_router, const T* __restrict__ bias, int n_tokens, int D, int n_route, int top) {
   extern __shared__ float smem[];
   float* hs = smem;                               // [TOK][D]
-  float* z = smem + TOK * D;                      // [TOK][n_route]
+  float* z = logits ? smem : smem + TOK * D;      // [TOK][n_route]
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int t0 = blockIdx.x * TOK, nt = min(TOK, n_tokens - t0);
   constexpr int V = Vec<T>::N;
   const bool vec = D % V == 0 && (reinterpret_cast<uintptr_t>(w_router) & 15) == 0;
-  if (vec && ldh % V == 0 && (reinterpret_cast<uintptr_t>(h) & 15) == 0) {
+  if (logits) {
+    for (int i = threadIdx.x; i < nt * n_route; i += blockDim.x)
+      z[i] = logits[(size_t)t0 * n_route + i] + (bias ? to_f<T>(bias[i % n_route]) : 0.f);
+  } else if (vec && ldh % V == 0 && (reinterpret_cast<uintptr_t>(h) & 15) == 0) {
     for (int i = threadIdx.x * V; i < TOK * D; i += blockDim.x * V) {
       const int tt = i / D, k = i - tt * D;
       float f[V];
@@ -221,7 +226,7 @@ moe_route_topk_kernel(int32_t* __restrict__ topk_idx, float* __restrict__ topk_w
     }
   }
   __syncthreads();
-  for (int e = warp; e < n_route; e += warps) {
+  for (int e = warp; !logits && e < n_route; e += warps) {
     const T* wr = w_router + (size_t)e * D;
     float acc[TOK];
 #pragma unroll
@@ -627,20 +632,20 @@ extern "C" int pg_moe_route_grouped(int32_t* topk_idx, float* topk_w, const void
   return PG_OK;
 }
 
-extern "C" int pg_moe_route_topk(int32_t* topk_idx, float* topk_w, const void* h, int ldh, const void* w_router, const void* bias,
-                                 int n_tokens, int D, int n_route, int top, int dtype, void* stream) {
+extern "C" int pg_moe_route_topk(int32_t* topk_idx, float* topk_w, const float* logits, const void* h, int ldh, const void* w_router,
+                                 const void* bias, int n_tokens, int D, int n_route, int top, int dtype, void* stream) {
   if (n_tokens <= 0) return PG_OK;
-  PG_REQUIRE(topk_idx && topk_w && h && w_router && top >= 1 && top <= n_route && n_route <= 4096,
+  PG_REQUIRE(topk_idx && topk_w && (logits || (h && w_router)) && top >= 1 && top <= n_route && n_route <= 4096,
              "moe_route_topk: top %d of %d routed outputs", top, n_route);
-  auto smem = [&](int tok) { return sizeof(float) * (size_t)tok * ((size_t)D + n_route); };
+  auto smem = [&](int tok) { return sizeof(float) * (size_t)tok * ((logits ? 0 : (size_t)D) + n_route); };
   PG_REQUIRE(smem(1) <= 200 * 1024, "moe_route_topk: D=%d with %d routed outputs does not fit shared memory", D, n_route);
   PG_DISPATCH_DTYPE(dtype, T, {
     if (n_tokens >= 296 && smem(8) <= 100 * 1024)
       return launch_pdl("moe_route_topk", moe_route_topk_kernel<T, 8>, dim3(cdiv(n_tokens, 8)), dim3(256), smem(8), (cudaStream_t)stream,
-                        topk_idx, topk_w, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens, D, n_route, top);
-    return launch_pdl("moe_route_topk", moe_route_topk_kernel<T, 1>, dim3(n_tokens), dim3(n_route >= 16 ? 512 : 256), smem(1),
-                      (cudaStream_t)stream, topk_idx, topk_w, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens, D,
-                      n_route, top);
+                        topk_idx, topk_w, logits, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens, D, n_route, top);
+    return launch_pdl("moe_route_topk", moe_route_topk_kernel<T, 1>, dim3(n_tokens), dim3(n_route >= 16 && !logits ? 512 : 256), smem(1),
+                      (cudaStream_t)stream, topk_idx, topk_w, logits, (const T*)h, ldh, (const T*)w_router, (const T*)bias, n_tokens,
+                      D, n_route, top);
   });
   return PG_OK;
 }

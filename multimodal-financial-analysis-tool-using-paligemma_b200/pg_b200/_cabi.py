@@ -148,7 +148,7 @@ SIGNATURES = {
     "pg_lru_conv": [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _vp],
     "pg_lru_ws_floats": [_i, _i, _i],
     "pg_lru_scan": [_vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _i, _i, _i, _i, _vp, _i, _i, _vp],
-    "pg_moe_route_topk": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "pg_moe_route_topk": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "pg_head_gemm_f32": [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "pg_latent_prep_ex": [_vp, _vp, _i, _i, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _i, _f, _f, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i,
                           _vp],

@@ -12,6 +12,10 @@ linear-attention scan the state-space layer runs on) (`run_gogivik`).
 norms, experts), Birizen (the decayed linear-attention scan) and Ninisun (the GeGLU feed-forward, the gated head norm)
 (`run_ranesun`).
 
+`bench.py --arch mutirax`: the Mutirax engine beside the models that hold its closest kernels: Birizen (latent attention, the
+decayed linear-attention scan, experts), Gogivik (convolutions over time, per-head norms and rotation, the state-space scan) and
+the MoE Mubasun (attention, norms) (`run_mutirax`).
+
 Timing: CUDA events on the launching stream, >= 3 warm-up steps, an L2-sized scratch write between timed steps.
 Roofline of an op = max(algorithmic FLOPs / measured bf16 peak, algorithmic bytes / measured copy bandwidth);
 `frac` = that time / measured time (1.0 = on the roofline)."""
@@ -1120,5 +1124,249 @@ def run_ranesun(sizes, steps: int, warmup: int, peaks: dict, prefill_tokens=2048
                                "distance_ratio": round(fb / fa, 2) if fa > 0 else None}
         row["like_for_like"] = cmpr
         result[name] = row
+    result["gpu_launches"] = int(cabi.launch_count() - launches0)
+    return result
+
+
+# ---------------------------------------------------------------------------------------------------------------
+MUTIRAX_SIZES = {
+    # latent layers, expert sizes and linear-attention heads as Birizen's; attention heads of the parallel layers as the Mubasun
+    # rows, beside a recurrent unit of the model's width; layers 0 and 1 run twice
+    "w1024": dict(width=1024, layers=4, heads=8, kv_heads=2, dim=128, vdim=128, rot_dim=64, q_rank=384, kv_rank=192, conv=4,
+                  lru_width=1024, lru_blocks=8, rank=16, ff=4096, experts=8, top=2, expert_ff=1024, streams=4, loop=(0, 2, 2),
+                  vocab=32000),
+    "w2048": dict(width=2048, layers=4, heads=16, kv_heads=4, dim=128, vdim=128, rot_dim=64, q_rank=768, kv_rank=192, conv=4,
+                  lru_width=2048, lru_blocks=16, rank=16, ff=8192, experts=16, top=2, expert_ff=2048, streams=4, loop=(0, 2, 2),
+                  vocab=32000),
+}
+
+
+def mutirax_config(s: dict) -> dict:
+    """latent + dense, parallel + experts, gla + experts, parallel + dense (every branch of the design is on the path)."""
+    latent = {"type": "latent_attention", "mixer": {
+        "heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "q_rank": s["q_rank"],
+        "kv_rank": s["kv_rank"], "scale": 1.0 / math.sqrt(s["dim"] + s["rot_dim"]),
+        "rot": {"dims": s["rot_dim"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+    parallel = {"type": "parallel", "mixer": {
+        "left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "conv": s["conv"],
+                 "scale": 1.0 / math.sqrt(s["dim"]), "rot": {"dims": s["dim"], "base": 10000.0}},
+        "right": {"width": s["lru_width"], "blocks": s["lru_blocks"], "conv": s["conv"]}}}
+    gla = {"type": "gla", "mixer": {"heads": s["heads"], "dim": s["dim"], "vdim": s["vdim"], "tau": 8.0}}
+    dense = {"kind": "dense", "ff": s["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    order = [(latent, dense), (parallel, moe), (gla, moe), (parallel, dense)]
+    return {"architecture": "Mutirax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "streams": s["streams"],
+            "residual_mult": 1.0, "layers": [dict(order[i % 4][0], mlp=order[i % 4][1]) for i in range(s["layers"])],
+            "loop": dict(zip(("start", "stop", "times"), s["loop"]))}
+
+
+def random_mutirax_weights(cfg: dict, s: dict, device, dtype, seed=0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(seed)
+    D, S, out = cfg["width"], cfg["streams"], {}
+
+    def lin(name, o, i):
+        out[name] = (torch.randn(o, i, generator=g, device=device) / math.sqrt(i)).to(dtype)
+
+    def vec(name, n, mean=0.0, std=0.1):
+        out[name] = (mean + std * torch.randn(n, generator=g, device=device)).to(dtype)
+
+    def norm(name):
+        vec(name, D, 1.0), vec(name + ".b", D)
+        out[name + ".alpha"] = torch.tensor(0.5, dtype=dtype, device=device)
+
+    def hyper(p):
+        vec(p + "in", S, 1.0 / S, 0.1), vec(p + "out", S, 0.5)
+        out[p + "mix"] = (torch.eye(S, device=device) * 0.8 + 0.2 / S + 0.05 * torch.randn(S, S, generator=g, device=device)).to(dtype)
+
+    out["embed"] = torch.randn(cfg["vocab"], D, generator=g, device=device).to(dtype)
+    lin("head", cfg["vocab"], D), norm("final.norm")
+    for i, L in enumerate(cfg["layers"]):
+        p, m, ml = f"l{i}.", L["mixer"], L["mlp"]
+        x = p + "mix."
+        norm(p + "norm1"), norm(p + "norm2"), hyper(p + "hc1."), hyper(p + "hc2.")
+        if L["type"] == "gla":
+            H, d, e, r = m["heads"], m["dim"], m["vdim"], s["rank"]
+            lin(x + "q", H * d, D), lin(x + "k", H * d, D), lin(x + "v", H * e, D), lin(x + "g", H * e, D), lin(x + "o", D, H * e)
+            vec(x + "norm", e, 1.0), lin(x + "a1", r, D), lin(x + "a2", H * d, r), vec(x + "a2.b", H * d, 0.0, 1.0)
+        elif L["type"] == "latent_attention":
+            H = m["heads"]
+            lin(x + "dq", m["q_rank"], D), vec(x + "dq.norm", m["q_rank"], 1.0), lin(x + "uq", H * (m["dim"] + m["rot_dim"]), m["q_rank"])
+            lin(x + "dkv", m["kv_rank"] + m["rot_dim"], D), vec(x + "dkv.norm", m["kv_rank"], 1.0)
+            lin(x + "uk", H * m["dim"], m["kv_rank"]), lin(x + "uv", H * m["vdim"], m["kv_rank"]), lin(x + "g", H, D)
+            lin(x + "o", D, H * m["vdim"])
+        else:
+            a, b = m["left"], m["right"]
+            nq, nk, w, bs = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], b["width"], b["width"] // b["blocks"]
+            l, r = x + "left.", x + "right."
+            lin(l + "q", nq, D), lin(l + "k", nk, D), vec(l + "q.norm", nq, 1.0), vec(l + "k.norm", nk, 1.0)
+            lin(l + "q.conv", nq, a["conv"]), lin(l + "k.conv", nk, a["conv"]), vec(l + "sink", a["heads"], 0.0, 1.0)
+            lin(l + "o", D, nq), vec(l + "out", D, 1.0), vec(r + "out", D, 1.0)
+            lin(r + "y", w, D), vec(r + "y.b", w), lin(r + "x", w, D), vec(r + "x.b", w), lin(r + "conv", w, b["conv"])
+            vec(r + "conv.b", w), vec(r + "lam", w, -3.0, 1.0), lin(r + "o", D, w)
+            for n in ("ra", "ri"):
+                lin(r + n, w, bs), vec(r + n + ".b", w)
+                out[r + n], out[r + n + ".b"] = out[r + n].view(b["blocks"], bs, bs), out[r + n + ".b"].view(b["blocks"], bs)
+        if ml["kind"] == "dense":
+            lin(p + "mlp.gate", ml["ff"], D), lin(p + "mlp.up", ml["ff"], D), lin(p + "mlp.down", D, ml["ff"])
+        else:
+            E = ml["router"]["experts"]
+            for e in range(E):
+                lin(f"{p}mlp.e{e}.gate", ml["expert"]["ff"], D), lin(f"{p}mlp.e{e}.up", ml["expert"]["ff"], D)
+                lin(f"{p}mlp.e{e}.down", D, ml["expert"]["ff"])
+            lin(p + "mlp.router", E, D), vec(p + "mlp.router.b", E)
+    return out
+
+
+def mutirax_work(s: dict, cfg: dict, T1: int, seqs: int) -> Dict[str, tuple]:
+    """name -> (FLOPs, bytes) of one step over `seqs` prompts of T1 tokens (bf16 operands, fp32 residual streams, fp32 scan
+    records, gates and states), summed over the layer runs."""
+    T, D, S, top = T1 * seqs, s["width"], s["streams"], s["top"]
+    P = T * top
+    w: Dict[str, List[float]] = {}
+
+    def add(name, flops, nbytes):
+        a = w.setdefault(name, [0.0, 0.0])
+        a[0] += flops
+        a[1] += nbytes
+
+    def gemm(name, N, K):
+        add(name, 2 * T * N * K, 2 * (T * K + N * K + T * N))
+
+    all_keys = seqs * T1 * (T1 + 1) // 2
+    # what the row kernel moves per column: streams in and out, the sublayer's rows, the next operand
+    move = {"connect": T * D * (8 * S + 2 + 2), "connect_pair": T * D * (8 * S + 4 + 2), "connect_experts": T * D * (8 * S + 2 * top + 2)}
+    add("connect", 0, T * D * (2 + 2))                                    # the first operand comes from the embedding row alone
+    written = False
+    for ri, L in enumerate(_looped_layers(s, cfg)):
+        m, ml = L["mixer"], L["mlp"]
+        if L["type"] == "gla":
+            H, d, e, r = m["heads"], m["dim"], m["vdim"], s["rank"]
+            rec = H * (3 * d + e)
+            gemm("proj", 2 * H * d + 2 * H * e + r, D)
+            add("gla_prep", 0, T * (2 * (H * (2 * d + e) + r) + 4 * rec))
+            add("gla", 4 * T * H * d * e, T * 4 * (rec + H * e))                         # fp32 FMAs, not tensor work
+            add("headnorm_gate", 0, T * H * e * (4 + 2 + 2))
+            gemm("o", D, H * e)
+            done = "connect"
+        elif L["type"] == "latent_attention":
+            H, d, rot, e, qr, kr = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"]
+            hq, hv, ldq = H * (d + rot), H * e, kr + rot
+            gemm("proj", qr + kr + rot + H, D)
+            add("latent_prep", 0, 2 * T * (2 * qr + 2 * (kr + rot)))
+            gemm("q_up", hq, qr)
+            add("q_absorb", 2 * T * H * d * kr, 2 * (T * hq + H * d * kr + T * H * ldq))
+            add("latent_attention", 2 * all_keys * H * (ldq + kr), 2 * T * H * (ldq + kr) + 2 * T * ldq)
+            add("v_up", 2 * T * H * kr * e, 2 * (T * H * kr + H * e * kr + T * hv))
+            gemm("o", D, hv)
+            done = "connect"
+        else:
+            a, b = m["left"], m["right"]
+            nq, nk, wd, bs = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], b["width"], b["width"] // b["blocks"]
+            gemm("proj", nq + nk + 2 * wd, D)
+            add("conv_qk_append", 0, 2 * T * (2 * nq + 3 * nk))
+            add("attention", 2 * all_keys * a["heads"] * 2 * a["dim"], 2 * T * (2 * nq + 2 * nk))
+            gemm("o", D, nq)
+            add("lru_conv", 0, T * wd * (2 + 2))
+            add("lru_gates", 2 * T * 2 * wd * bs, T * wd * (2 + 8) + 2 * 2 * wd * bs)
+            add("lru_scan", 0, T * wd * (8 + 2 + 2 + 2))                                # gates, u, y in; the product out: once each
+            gemm("o", D, wd)
+            add("conv_state", 0, seqs * (a["conv"] - 1) * (nq + nk + wd) * (2 + 4))
+            done = "connect_pair"
+        add(done, 0, move[done] - (0 if written else 4 * S * T * D - 2 * T * D))        # the first sum reads embedding rows, not streams
+        written = True
+        if ml["kind"] == "dense":
+            F = ml["ff"]
+            gemm("gate_up", 2 * F, D)
+            add("glu", 0, T * F * (4 + 2))
+            gemm("down", D, F)
+            done = "connect"
+        else:
+            E, F = ml["router"]["experts"], ml["expert"]["ff"]
+            add("moe_route", 2 * T * D * E, 2 * T * D)
+            add("moe_sort", 0, 4 * 3 * P)
+            add("moe_gather", 0, 2 * 2 * P * D)
+            add("moe_gate_up", 2 * P * D * 2 * F, 2 * (P * D + E * 2 * F * D + P * F))
+            add("moe_down", 2 * P * F * D, 2 * (P * F + E * F * D + P * D))
+            done = "connect_experts"
+        if ri + 1 < s["layers"] + (s["loop"][1] - s["loop"][0]) * (s["loop"][2] - 1):   # the last sum is of the wanted rows alone
+            add(done, 0, move[done])
+    add("head", 2 * seqs * D * s["vocab"], 2 * D * s["vocab"])
+    return {k: (v[0], v[1]) for k, v in w.items()}
+
+
+def _mutirax_decode_bytes(s: dict, cfg: dict, B: int) -> float:
+    """Weight bytes one decode step of B tokens must stream (experts: at most B * top of them per MoE layer run)."""
+    D, n = s["width"], 0.0
+    for L in _looped_layers(s, cfg):
+        m, ml = L["mixer"], L["mlp"]
+        if L["type"] == "gla":
+            n += D * (m["heads"] * (2 * m["dim"] + 3 * m["vdim"]) + s["rank"]) + m["heads"] * m["dim"] * s["rank"]
+        elif L["type"] == "latent_attention":
+            H = m["heads"]
+            n += D * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + H + H * m["vdim"]) + m["q_rank"] * H * (m["dim"] + m["rot_dim"])
+            n += H * m["kv_rank"] * (m["dim"] + m["vdim"])
+        else:
+            a, b = m["left"], m["right"]
+            n += D * (a["dim"] * (2 * a["heads"] + a["kv_heads"]) + 3 * b["width"]) + 2 * b["width"] * (b["width"] // b["blocks"])
+        n += 3 * D * ml["ff"] if ml["kind"] == "dense" else min(s["experts"], B * s["top"]) * 3 * D * s["expert_ff"] + D * s["experts"]
+    return 2.0 * (n + D * s["vocab"])
+
+
+MUTIRAX_LIKE_BIRIZEN = [("gla", "lightning"), ("gla_prep", "lightning_prep"), ("headnorm_gate", "headnorm_gate"),
+                        ("latent_prep", "latent_prep"), ("q_up", "q_up"), ("q_absorb", "q_absorb"), ("latent_attention", "latent_attention"),
+                        ("v_up", "v_up_gate"), ("lru_gates", "q_absorb"), ("moe_route", "moe_route"), ("moe_sort", "moe_sort"),
+                        ("moe_gather", "moe_gather"), ("moe_gate_up", "moe_gate_up"), ("moe_down", "moe_down"),
+                        ("connect_experts", "post_norm"), ("proj", "proj"), ("o", "o"), ("head", "head")]
+MUTIRAX_LIKE_GOGIVIK = [("conv_qk_append", "headnorm_rotary_append"), ("lru_conv", "norm_conv"), ("lru_scan", "ssm_scan"),
+                        ("connect", "norm_conv"), ("glu", "relu2"), ("down", "down")]
+MUTIRAX_LIKE_MUBASUN = [("attention", "attention"), ("connect_pair", "norm"), ("gate_up", "dense_up")]
+
+
+@torch.no_grad()
+def run_mutirax(sizes, steps: int, warmup: int, peaks: dict, prefill_tokens=2048, prefill_seqs=4, context=1024,
+                decode_batches=(1, 8), alone: bool = False) -> dict:
+    from .birizen import BirizenEngine
+    from .gogivik import GogivikEngine
+    from .mubasun import MubasunEngine
+    from .mutirax import MutiraxEngine
+    dev, dtype = torch.device("cuda:0"), torch.bfloat16
+    timer = _Timer()
+    result = {}
+    launches0 = cabi.launch_count()
+    pool = (max(max(decode_batches), prefill_seqs) + 1) * (max(prefill_tokens, context) + 256)
+
+    def measure(cls, cfg, weights, size, work, decode_bytes):
+        eng = cls(cfg, weights, device=dev, dtype=dtype, kv_pool_tokens=pool)
+        out = _measure_ragged(eng, size["vocab"], timer, steps, warmup, peaks, work(size, cfg, prefill_tokens, prefill_seqs),
+                              decode_bytes, prefill_tokens, prefill_seqs, context, decode_batches)
+        del eng
+        torch.cuda.empty_cache()
+        return out
+
+    for name in sizes:
+        s, bs_, gs_, ms_ = MUTIRAX_SIZES[name], BIRIZEN_SIZES[name], GOGIVIK_SIZES[name], SIZES[name]
+        cfg, bcfg, gcfg, mcfg = mutirax_config(s), birizen_config(bs_), gogivik_config(gs_), mubasun_config(ms_)
+        row = {"size": s}
+        row.update(measure(MutiraxEngine, cfg, random_mutirax_weights(cfg, s, dev, dtype), s, mutirax_work,
+                           lambda B: _mutirax_decode_bytes(s, cfg, B)))
+        result[name] = row
+        if alone:
+            continue
+        row["birizen_equal_size"] = measure(BirizenEngine, bcfg, random_birizen_weights(bcfg, dev, dtype), bs_, birizen_work,
+                                            lambda B: _birizen_decode_bytes(bs_, bcfg, B))
+        row["gogivik_equal_size"] = measure(GogivikEngine, gcfg, random_gogivik_weights(gcfg, dev, dtype), gs_, gogivik_work,
+                                            lambda B: _gogivik_decode_bytes(gs_, gcfg))
+        row["mubasun_equal_size"] = measure(MubasunEngine, mcfg, random_mubasun_weights(mcfg, dev, dtype), ms_, mubasun_work,
+                                            lambda B: _decode_bytes(ms_, mcfg, B))
+        cmpr = {}
+        for like, other in ((MUTIRAX_LIKE_BIRIZEN, "birizen_equal_size"), (MUTIRAX_LIKE_GOGIVIK, "gogivik_equal_size"),
+                            (MUTIRAX_LIKE_MUBASUN, "mubasun_equal_size")):
+            ops = row[other]["prefill_ops"]
+            for a, bname in like:
+                if a in row["prefill_ops"] and bname in ops:
+                    fa, fb = row["prefill_ops"][a]["frac"], ops[bname]["frac"]
+                    cmpr[a] = {"frac": fa, "like": f"{bname} ({other.split('_')[0]})", "like_frac": fb,
+                               "distance_ratio": round(fb / fa, 2) if fa > 0 else None}
+        row["like_for_like"] = cmpr
     result["gpu_launches"] = int(cabi.launch_count() - launches0)
     return result

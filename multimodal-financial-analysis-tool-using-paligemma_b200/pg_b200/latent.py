@@ -20,6 +20,8 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Optional
 
+import torch
+
 from . import _cabi as cabi
 from ._cabi import ptr
 from .ragged_engine import RotaryCfg, StepInputs, _stack_rows, rotary_pairs

@@ -181,6 +181,7 @@ class MutiraxEngine(LatentAttentionMixin, RaggedEngine):
         self.runs = self.cfg.runs()
         self.needs_segments = any(lc.kind != "latent_attention" for lc in self.cfg.layers)
         self.lru_impl = 0               # recurrent unit: 0 picks, 1 token by token, 2 chunked
+        self.route_gemm_min = 256       # tokens from which the router's logits are a GEMM of their own
         self._repack(weights)
         L_ = cabi.lib()
         for w, lc in zip(self.layers, self.cfg.layers):     # prompt portions of layers whose sizes the tensor-core kernel takes
@@ -275,14 +276,14 @@ class MutiraxEngine(LatentAttentionMixin, RaggedEngine):
         w["proj"], w["at"] = _stack_rows([("q", W(l + "q", (nq, D))), ("k", W(l + "k", (nk, D))), ("x", W(r + "x", (rt.width, D))),
                                           ("y", W(r + "y", (rt.width, D)))], self.device, self.dtype)
         at = w["at"]
-        conv = torch.zeros((lf.taps, at["k"] + nk), dtype=f32, device=self.device)      # [taps][columns], the current token last
-        conv[:, :nq] = W(l + "q.conv", (nq, lf.taps), f32).T
-        conv[:, at["k"]:] = W(l + "k.conv", (nk, lf.taps), f32).T
+        conv = torch.zeros((lf.taps, at["k"] + nk), dtype=self.dtype, device=self.device)   # [taps][columns], the current token last
+        conv[:, :nq] = W(l + "q.conv", (nq, lf.taps)).T
+        conv[:, at["k"]:] = W(l + "k.conv", (nk, lf.taps)).T
         w.update(conv=conv, q_norm=W(l + "q.norm", (nq,)), k_norm=W(l + "k.norm", (nk,)), sink=W(l + "sink", (lf.heads,), f32),
                  freq=rotary_pairs(lf.rot).to(self.device) if lf.rot else None, o=W(l + "o", (D, nq)), left_out=W(l + "out", (D,)))
         gates = torch.cat([W(r + "ra", (rt.blocks, bs, bs)), W(r + "ri", (rt.blocks, bs, bs))], 1).contiguous()
         w.update(x_b=W(r + "x.b", (rt.width,)), y_b=W(r + "y.b", (rt.width,)), gates=gates,
-                 r_conv=W(r + "conv", (rt.width, rt.taps), f32).T.contiguous(), r_conv_b=W(r + "conv.b", (rt.width,)),
+                 r_conv=W(r + "conv", (rt.width, rt.taps)).T.contiguous(), r_conv_b=W(r + "conv.b", (rt.width,)),
                  ra_b=W(r + "ra.b", (rt.blocks, bs)).reshape(-1), ri_b=W(r + "ri.b", (rt.blocks, bs)).reshape(-1),
                  lam=W(r + "lam", (rt.width,), f32), r_o=W(r + "o", (D, rt.width)), right_out=W(r + "out", (D,)),
                  conv_len=max(lf.taps, rt.taps) - 1, conv_cols=at["x"] + rt.width)
@@ -414,9 +415,14 @@ class MutiraxEngine(LatentAttentionMixin, RaggedEngine):
     def _moe(self, h, ml: MlpCfg, w: dict) -> dict:
         T, D = h.shape
         idx, wts = self._new(T * ml.top, dtype=torch.int32), self._new(T * ml.top, dtype=torch.float32)
+        L, st, z = cabi.lib(), cabi.stream(), None
         with self._tm("moe_route"):
-            cabi.check(cabi.lib().pg_moe_route_topk(ptr(idx), ptr(wts), ptr(h), h.stride(0), ptr(w["router"]), ptr(w["router_b"]), T, D,
-                                                    ml.experts, ml.top, self.dt, cabi.stream()), "moe_route_topk")
+            if T >= self.route_gemm_min and self.dtype != torch.float32 and D % 8 == 0 and ml.experts % 8 == 0:
+                z = self._new(T, ml.experts, dtype=torch.float32)       # prompt portions: the fp32 logits on the tensor cores
+                cabi.check(L.pg_head_gemm_f32(ptr(z), ml.experts, 0, ptr(h), h.stride(0), 0, ptr(w["router"]), T, 1, ml.experts, D, 0,
+                                              ptr(self.err_flag), self.dt, st), "router logits")
+            cabi.check(L.pg_moe_route_topk(ptr(idx), ptr(wts), ptr(z), ptr(h), h.stride(0), ptr(w["router"]), ptr(w["router_b"]), T, D,
+                                           ml.experts, ml.top, self.dt, st), "moe_route_topk")
         y, pos = self._moe_experts(h, idx, ml.experts, ml.top, ml.ff, w["gu"], w["dn"], cabi.GLU_SILU)
         return {"experts": (y, pos, wts, ml.top)}
 
