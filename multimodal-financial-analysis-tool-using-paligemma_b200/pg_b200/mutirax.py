@@ -106,13 +106,13 @@ class LayerCfg:
 def _conv_attn_cfg(i: int, m: Mapping) -> ConvAttnCfg:
     heads, dim, rot = int(m["heads"]), int(m["dim"]), m.get("rot")
     a = ConvAttnCfg(heads=heads, kv_heads=int(m.get("kv_heads", heads)), dim=dim, scale=float(m["scale"]), taps=int(m["conv"]),
-                    rot=RotaryCfg(int(rot["dims"]), float(rot["base"]), rot.get("scaling")) if rot and int(rot["dims"]) else None)
+                    rot=RotaryCfg(int(rot["dims"]), float(rot["base"])) if rot and int(rot["dims"]) else None)
     if a.heads % a.kv_heads or a.taps < 1:
         raise ValueError(f"layer {i}: {a.heads} heads over {a.kv_heads} key heads, {a.taps} taps")
     if int(m.get("vdim", dim)) != dim:
         raise ValueError(f"layer {i}: the values are the keys, so vdim {m['vdim']} must be dim {dim}")
-    if a.rot and (a.rot.dims % 2 or a.rot.dims > dim):
-        raise ValueError(f"layer {i}: {a.rot.dims} rotated columns of {dim}")
+    if a.rot and (a.rot.dims % 2 or a.rot.dims > dim or rot.get("scaling")):
+        raise ValueError(f"layer {i}: {a.rot.dims} rotated columns of {dim}, frequency scaling {rot.get('scaling')}")
     return a
 
 

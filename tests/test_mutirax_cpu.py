@@ -52,6 +52,9 @@ def test_config_rejects_what_the_design_does_not_have():
     apart = par()
     apart["mixer"]["left"]["vdim"] = 6                          # the values are the keys
     bad([O.layer(apart)])
+    scaled = par()
+    scaled["mixer"]["left"]["rot"]["scaling"] = {"factor": 2.0}   # frequencies are scaled in the latent mixer alone
+    bad([O.layer(scaled)])
     turned = O.latent(heads=1, dim=4, rot_dim=4, vdim=4, q_rank=4, kv_rank=4)
     turned["mixer"]["rot"]["dims"] = 2                          # the rotated part is rotated whole
     bad([O.layer(turned)])
